@@ -938,7 +938,10 @@ MG_API int mg_attention_wide(const void* q, int q_stride, const void* k_pages, c
     const bool aligned = d % 8 == 0 && dv % 8 == 0 && q_stride % 8 == 0 && (gate == nullptr || gate_stride % 2 == 0) &&
                          ((uintptr_t)q % 16 == 0) && ((uintptr_t)k_pages % 16 == 0) && ((uintptr_t)out % 4 == 0) &&
                          ((uintptr_t)gate % 4 == 0);
-    const int dpad = (d + 15) / 16 * 16;
+    // the values' columns, padded, in four equal parts of whole pairs of 8-column tiles; the key rows in shared memory are
+    // padded (with zeros) to hold them all
+    const int dv_pad = dv <= 64 ? 64 : dv <= 128 ? 128 : dv <= 256 ? 256 : 512;
+    const int dpad = (d + 15) / 16 * 16 > dv_pad ? (d + 15) / 16 * 16 : dv_pad;
     const size_t smem = ((size_t)(WIDE_ROWS + 2 * KB) * (dpad + PAD) + WIDE_ROWS * (KB + PAD)) * sizeof(bf16) + 4 * WIDE_ROWS * sizeof(float);
     if (!aligned || dv > 512 || smem > 227 * 1024 || n_kv_head > 65535) return MG_ERR_UNSUPPORTED;
     AttnParams p;
@@ -960,11 +963,8 @@ MG_API int mg_attention_wide(const void* q, int q_stride, const void* k_pages, c
         MG_REQUIRE(req_q_start && req_q_len && n_tiles > 0, "attention (wide rows): no tiles");
     }
     cudaStream_t s = (cudaStream_t)stream;
-    // the values' columns, padded, in four equal parts of whole pairs of 8-column tiles; padded columns lie inside
-    // the padded key row (dv <= d) or, beyond it, in the row's padding and the next row: they are never stored
-    if (dv <= 64 && dpad >= 64) return launch_wide<16>(p, single_tokens, n_tiles, dpad, smem, s);
-    if (dv <= 128 && dpad >= 128) return launch_wide<32>(p, single_tokens, n_tiles, dpad, smem, s);
-    if (dv <= 256 && dpad >= 256) return launch_wide<64>(p, single_tokens, n_tiles, dpad, smem, s);
-    if (dpad >= 512) return launch_wide<128>(p, single_tokens, n_tiles, dpad, smem, s);
-    return MG_ERR_UNSUPPORTED;
+    if (dv_pad == 64) return launch_wide<16>(p, single_tokens, n_tiles, dpad, smem, s);
+    if (dv_pad == 128) return launch_wide<32>(p, single_tokens, n_tiles, dpad, smem, s);
+    if (dv_pad == 256) return launch_wide<64>(p, single_tokens, n_tiles, dpad, smem, s);
+    return launch_wide<128>(p, single_tokens, n_tiles, dpad, smem, s);
 }

@@ -3,9 +3,11 @@
 //
 //   route:   z = W_r h (32-bit), the `top` largest z choose experts (ties: the lower index), their
 //            weights are softmax over the chosen z alone; optionally g = sigmoid(w_g . h), one number
-//            per token (the gate of an expert that every token uses).
+//            per token (the gate of an expert that every token uses; such experts can join the chosen ones as
+//            further entries of every token, g their weight).
 //   group:   entry (token, k) -> a slot; the slots of one expert are contiguous and in entry order.
-//   experts: H[slot] = silu(W_gate[e] h) * (W_up[e] h);  Y[slot] = weight[slot] * W_down[e] H[slot]  (32-bit)
+//   experts: H[slot] = silu(W_gate[e] h) * (W_up[e] h), or act(W_up[e] h) for experts without a gate;
+//            Y[slot] = weight[slot] * W_down[e] H[slot]  (32-bit)
 //   combine: x[token] += sum_k Y[slot of (token, k)], k in order: the same sum whatever the grouping.
 //
 // Nothing here depends on the host knowing how many tokens an expert got: grids are sized for the
@@ -48,32 +50,39 @@ template <typename T>
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ w_gate,
                  const int* __restrict__ positions, int* __restrict__ ids, float* __restrict__ weights,
-                 float* __restrict__ gate, int n_tokens, int width, int n_experts, int top) {
-    extern __shared__ float z[];                           // [n_experts]
+                 float* __restrict__ gate, int n_tokens, int width, int n_experts, int top, int always) {
+    extern __shared__ float z[];                           // [n_experts], then the gate
     pdl_trigger();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int token = blockIdx.x;
     if (positions != nullptr && positions[token] < 0) {    // padding of a fixed-size batch: no expert
-        for (int k = threadIdx.x; k < top; k += blockDim.x) {
-            ids[(size_t)token * top + k] = -1;
-            weights[(size_t)token * top + k] = 0.f;
+        for (int k = threadIdx.x; k < top + always; k += blockDim.x) {
+            ids[(size_t)token * (top + always) + k] = -1;
+            weights[(size_t)token * (top + always) + k] = 0.f;
         }
         if (gate != nullptr && threadIdx.x == 0) gate[token] = 0.f;
         return;
     }
     const T* row = h + (size_t)token * width;
     const bool vec = width % 4 == 0 && ((uintptr_t)w_router % 16 == 0) && (w_gate == nullptr || (uintptr_t)w_gate % 16 == 0);
-    const int rows = n_experts + (gate != nullptr ? 1 : 0);
+    const int rows = n_experts + (w_gate != nullptr ? 1 : 0);
+    ids += (size_t)token * (top + always), weights += (size_t)token * (top + always);
     for (int e = warp; e < rows; e += ROUTE_WARPS) {
         const float dot = route_dot(row, e < n_experts ? w_router + (size_t)e * width : w_gate, width, lane, vec);
         if (lane == 0) {
             if (e < n_experts) z[e] = dot;
-            else gate[token] = 1.0f / (1.0f + expf(-dot));
+            else z[e] = 1.0f / (1.0f + expf(-dot));
         }
     }
     __syncthreads();
     if (warp != 0) return;
+    if (gate != nullptr && lane == 0) gate[token] = z[n_experts];
+    // experts that every token uses, behind the chosen ones
+    for (int k = lane; k < always; k += 32) {
+        ids[top + k] = n_experts + k;
+        weights[top + k] = w_gate != nullptr ? z[n_experts] : 1.f;
+    }
     // the `top` largest, one after the other; every lane looks at a share of the experts
     float z_max = 0.f, sum = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -94,14 +103,14 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
         const float p = expf(best - z_max);
         sum += p;
         if (lane == 0) {
-            ids[(size_t)token * top + k] = best_e;
-            weights[(size_t)token * top + k] = p;
+            ids[k] = best_e;
+            weights[k] = p;
             z[best_e] = -INFINITY;
         }
         __syncwarp();
     }
     const float inv = 1.0f / sum;
-    for (int k = lane; k < top; k += 32) weights[(size_t)token * top + k] *= inv;
+    for (int k = lane; k < top; k += 32) weights[k] *= inv;
 }
 
 // ---- router with scores per expert, a correction for the choice, and groups --------------------------
@@ -296,13 +305,18 @@ __device__ __forceinline__ float gated_value(int act, float limit, float g, floa
     return silu(g) * u;
 }
 
-// GLU = true:  out[slot, n] = silu(a . w[e][n]) * (a . w[e][inner + n]),  a = x[token of slot]   (T out)
-// GLU = false: out[slot, n] = scale[entry of slot] * (a . w[e][n]),       a = x[slot]            (32-bit out)
-template <typename T, bool GLU>
+// A unit without a gate: its one hidden feature z, by `act` (0: max(z, 0)^2, 1: gelu_tanh(z), 2: silu(z)).
+__device__ __forceinline__ float plain_value(int act, float z) { return act == 0 ? relu_sq(z) : act == 1 ? gelu_tanh(z) : silu(z); }
+
+// FORM 1 (gated): out[slot, n] = silu(a . w[e][n]) * (a . w[e][inner + n]),  a = x[token of slot]   (T out)
+// FORM 2 (plain): out[slot, n] = act(a . w[e][n]),                           a = x[token of slot]   (T out)
+// FORM 0 (out):   out[slot, n] = scale[entry of slot] * (a . w[e][n]),       a = x[slot]            (32-bit out)
+template <typename T, int FORM>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, long long w_expert_stride,
                 const int* __restrict__ offsets, const int* __restrict__ slot_entry, int top,
                 const float* __restrict__ scale, void* __restrict__ out, int N, int K, int x_rows, int act, float limit) {
+    constexpr bool GLU = FORM == 1;
     __shared__ float as[BK][BM + 4];
     __shared__ float ws[BK][BN + 4];
     __shared__ float us[GLU ? BK : 1][BN + 4];
@@ -319,7 +333,7 @@ moe_gemm_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, long 
         int r = -1;
         if (m0 + tid < count) {
             const int slot = first + m0 + tid;
-            r = GLU ? slot_entry[slot] / top : slot;
+            r = FORM != 0 ? slot_entry[slot] / top : slot;
             if (!MG_GUARDED(moe, MG_GUARD_ROW, r, x_rows)) r = -1;
         }
         row_of[tid] = r;
@@ -372,13 +386,15 @@ moe_gemm_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, long 
         const int m = m0 + tr * TM + i;
         if (m >= count) continue;
         const size_t slot = (size_t)first + m;
-        const float sc = GLU ? 1.f : scale[slot_entry[slot]];
+        const float sc = FORM != 0 ? 1.f : scale[slot_entry[slot]];
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int n = n0 + tc * TN + j;
             if (n >= N) continue;
             if constexpr (GLU)
                 reinterpret_cast<T*>(out)[slot * N + n] = from_float<T>(gated_value(act, limit, acc[i][j], acc_u[i][j]));
+            else if constexpr (FORM == 2)
+                reinterpret_cast<T*>(out)[slot * N + n] = from_float<T>(plain_value(act, acc[i][j]));
             else
                 reinterpret_cast<float*>(out)[slot * N + n] = acc[i][j] * sc;
         }
@@ -415,11 +431,12 @@ __device__ __forceinline__ void copy16_async(bf16* dst, const bf16* src, bool re
 // matrices is in flight when the work is nothing but reading them.
 // NS: shared-memory buffers that take turns (NS - 1 tiles are in flight while one is multiplied): two
 // where many CTAs share an SM, four where a CTA does little but wait for its matrix.
-template <bool GLU, int MB, int NS>
+template <int FORM, int MB, int NS>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__ w, long long w_expert_stride,
                     const int* __restrict__ offsets, const int* __restrict__ slot_entry, int top,
                     const float* __restrict__ scale, void* __restrict__ out, int N, int K, int x_rows, int act, float limit) {
+    constexpr bool GLU = FORM == 1;
     extern __shared__ __align__(16) uint8_t moe_smem[];
     bf16* as = reinterpret_cast<bf16*>(moe_smem);          // [NS][MT * MLD]
     bf16* bs = as + NS * MT * MLD;                         // [NS][MB * MLD]
@@ -438,7 +455,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
         int r = -1;
         if (m0 + tid < count) {
             const int slot = first + m0 + tid;
-            r = GLU ? slot_entry[slot] / top : slot;
+            r = FORM != 0 ? slot_entry[slot] / top : slot;
             if (!MG_GUARDED(moe, MG_GUARD_ROW, r, x_rows)) r = -1;
         }
         row_of[tid] = r;
@@ -544,6 +561,18 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
                         if (n + 1 < N) o[1] = __float2bfloat16_rn(v1);
                     }
                 }
+            } else if (FORM == 2) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const int n = n0 + wc * 64 + j * 8 + 2 * (lane & 3);
+                    const float v0 = plain_value(act, acc[i][j][2 * half]), v1 = plain_value(act, acc[i][j][2 * half + 1]);
+                    bf16* o = reinterpret_cast<bf16*>(out) + slot * N + n;
+                    if (n + 1 < N && (N & 1) == 0) *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, v1);
+                    else {
+                        if (n < N) o[0] = __float2bfloat16_rn(v0);
+                        if (n + 1 < N) o[1] = __float2bfloat16_rn(v1);
+                    }
+                }
             } else {
                 const float sc = scale[slot_entry[slot]];
 #pragma unroll
@@ -596,24 +625,26 @@ __global__ void glu_kernel(const T* __restrict__ gu, const float* __restrict__ s
 }  // namespace
 
 // h: [n_tokens, width] (bfloat16 if is_bf16 else 32-bit); w_router: [n_experts, width] and w_gate:
-// [width] (null: no gate), 32-bit; positions: [n_tokens] or null; ids, weights: [n_tokens, top];
-// gate: [n_tokens] or null.
+// [width] (null: no gate), 32-bit; positions: [n_tokens] or null; ids, weights: [n_tokens, top + always]: behind a
+// token's chosen experts the experts n_experts .. n_experts + always - 1, which every token uses, with the gate's value
+// (1 without a gate) as their weight; gate: [n_tokens] or null.
 MG_API int mg_moe_route(const void* h, const float* w_router, const float* w_gate, const int* positions, int* ids,
-                        float* weights, float* gate, int n_tokens, int width, int n_experts, int top, int is_bf16,
-                        void* stream) {
+                        float* weights, float* gate, int n_tokens, int width, int n_experts, int top, int always,
+                        int is_bf16, void* stream) {
     if (n_tokens == 0) return MG_OK;
     MG_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top > 0 && top <= n_experts, "moe route: bad sizes");
-    MG_REQUIRE((w_gate == nullptr) == (gate == nullptr), "moe route: a gate wants its weights and its output");
-    const size_t smem = (size_t)n_experts * sizeof(float);
+    MG_REQUIRE(gate == nullptr || w_gate != nullptr, "moe route: a gate wants its weights");
+    MG_REQUIRE(always >= 0 && (w_gate == nullptr || gate != nullptr || always > 0), "moe route: a gate that nothing takes");
+    const size_t smem = (size_t)(n_experts + 1) * sizeof(float);
     MG_REQUIRE(smem <= 48 * 1024, "moe route: too many experts (%d)", n_experts);
     const dim3 grid(n_tokens), block(32 * ROUTE_WARPS);
     cudaError_t e;
     if (is_bf16)
         e = mg_launch(moe_route_kernel<bf16>, grid, block, smem, (cudaStream_t)stream, true, (const bf16*)h, w_router,
-                      w_gate, positions, ids, weights, gate, n_tokens, width, n_experts, top);
+                      w_gate, positions, ids, weights, gate, n_tokens, width, n_experts, top, always);
     else
         e = mg_launch(moe_route_kernel<float>, grid, block, smem, (cudaStream_t)stream, true, (const float*)h, w_router,
-                      w_gate, positions, ids, weights, gate, n_tokens, width, n_experts, top);
+                      w_gate, positions, ids, weights, gate, n_tokens, width, n_experts, top, always);
     MG_LAUNCHED(e, "moe route");
     return MG_OK;
 }
@@ -657,20 +688,21 @@ MG_API int mg_moe_group(const int* ids, int n_entries, int n_experts, int* offse
     return MG_OK;
 }
 
-// act, limit: the gated product of the first product's two halves (see gated_value).
-// glu = 1: x [x_rows, ldx] gathered by token, w [n_experts, 2 N, K], out [n_entries, N] in the inputs' type.
-// glu = 0: x [n_entries, ldx] by slot, w [n_experts, N, K], scale [n_entries] by entry, out [n_entries, N] 32-bit.
+// act, limit: what the first product's epilogue computes (gated_value, plain_value).
+// form 1 (gated): x [x_rows, ldx] gathered by token, w [n_experts, 2 N, K], out [n_entries, N] in the inputs' type.
+// form 2 (plain): the same with w [n_experts, N, K].
+// form 0 (out):   x [n_entries, ldx] by slot, w [n_experts, N, K], scale [n_entries] by entry, out [n_entries, N] 32-bit.
 // max_rows: the most slots one expert can have (the tokens of the step).
 MG_API int mg_moe_gemm(const void* x, int ldx, const void* w, const int* offsets, const int* slot_entry, int top,
-                       const float* scale, void* out, int n_experts, int max_rows, int N, int K, int x_rows, int glu,
+                       const float* scale, void* out, int n_experts, int max_rows, int N, int K, int x_rows, int form,
                        int is_bf16, int act, float limit, void* stream) {
     if (max_rows == 0) return MG_OK;
-    MG_REQUIRE(n_experts > 0 && n_experts <= 65535 && max_rows > 0 && N > 0 && K > 0 && ldx >= K && top > 0,
+    MG_REQUIRE(n_experts > 0 && n_experts <= 65535 && max_rows > 0 && N > 0 && K > 0 && ldx >= K && top > 0 && form >= 0 && form <= 2,
                "moe gemm: bad sizes");
-    MG_REQUIRE(glu || scale != nullptr, "moe gemm: the second product wants the entries' weights");
+    MG_REQUIRE(form != 0 || scale != nullptr, "moe gemm: the second product wants the entries' weights");
     const dim3 grid(ceil_div(N, BN), ceil_div(max_rows, BM), n_experts), block(256);
     MG_REQUIRE(grid.y <= 65535, "moe gemm: too many rows");
-    const long long stride = (long long)(glu ? 2 : 1) * N * K;
+    const long long stride = (long long)(form == 1 ? 2 : 1) * N * K;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
     const bool tensor_cores = is_bf16 && K % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
@@ -678,45 +710,32 @@ MG_API int mg_moe_gemm(const void* x, int ldx, const void* w, const int* offsets
     if (tensor_cores) {
         const bool few = max_rows <= MT;                    // few tokens: narrower tiles, more CTAs
         const int mb = few ? 64 : 128;
-        const dim3 tgrid(ceil_div(N, glu ? mb / 2 : mb), ceil_div(max_rows, MT), n_experts);
+        const dim3 tgrid(ceil_div(N, form == 1 ? mb / 2 : mb), ceil_div(max_rows, MT), n_experts);
+        using Kernel = void (*)(const bf16*, int, const bf16*, long long, const int*, const int*, int, const float*, void*, int, int,
+                                int, int, float);
+        static const Kernel wide[3] = {moe_gemm_mma_kernel<0, 128, 2>, moe_gemm_mma_kernel<1, 128, 2>, moe_gemm_mma_kernel<2, 128, 2>};
+        static const Kernel narrow[3] = {moe_gemm_mma_kernel<0, 64, 4>, moe_gemm_mma_kernel<1, 64, 4>, moe_gemm_mma_kernel<2, 64, 4>};
         static bool configured = false;
         if (!configured) {
-            e = cudaFuncSetAttribute(moe_gemm_mma_kernel<true, 128, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)moe_mma_smem(128, 2));
-            if (e == cudaSuccess)
-                e = cudaFuncSetAttribute(moe_gemm_mma_kernel<false, 128, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)moe_mma_smem(128, 2));
-            if (e == cudaSuccess)
-                e = cudaFuncSetAttribute(moe_gemm_mma_kernel<true, 64, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)moe_mma_smem(64, 4));
-            if (e == cudaSuccess)
-                e = cudaFuncSetAttribute(moe_gemm_mma_kernel<false, 64, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)moe_mma_smem(64, 4));
-            MG_LAUNCHED(e, "moe gemm (shared memory)");
+            for (int f = 0; f < 3; ++f) {
+                e = cudaFuncSetAttribute((const void*)wide[f], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)moe_mma_smem(128, 2));
+                if (e == cudaSuccess)
+                    e = cudaFuncSetAttribute((const void*)narrow[f], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)moe_mma_smem(64, 4));
+                MG_LAUNCHED(e, "moe gemm (shared memory)");
+            }
             configured = true;
         }
-        const bf16* xb = (const bf16*)x;
-        const bf16* wb = (const bf16*)w;
-        if (glu && few)
-            e = mg_launch(moe_gemm_mma_kernel<true, 64, 4>, tgrid, dim3(128), moe_mma_smem(64, 4), s, true, xb, ldx, wb, stride,
-                          offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-        else if (glu)
-            e = mg_launch(moe_gemm_mma_kernel<true, 128, 2>, tgrid, dim3(128), moe_mma_smem(128, 2), s, true, xb, ldx, wb, stride,
-                          offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-        else if (few)
-            e = mg_launch(moe_gemm_mma_kernel<false, 64, 4>, tgrid, dim3(128), moe_mma_smem(64, 4), s, true, xb, ldx, wb, stride,
-                          offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-        else
-            e = mg_launch(moe_gemm_mma_kernel<false, 128, 2>, tgrid, dim3(128), moe_mma_smem(128, 2), s, true, xb, ldx, wb, stride,
-                          offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-    } else if (is_bf16 && glu)
-        e = mg_launch(moe_gemm_kernel<bf16, true>, grid, block, 0, s, true, (const bf16*)x, ldx, (const bf16*)w, stride,
-                      offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-    else if (is_bf16)
-        e = mg_launch(moe_gemm_kernel<bf16, false>, grid, block, 0, s, true, (const bf16*)x, ldx, (const bf16*)w, stride,
-                      offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-    else if (glu)
-        e = mg_launch(moe_gemm_kernel<float, true>, grid, block, 0, s, true, (const float*)x, ldx, (const float*)w, stride,
-                      offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
-    else
-        e = mg_launch(moe_gemm_kernel<float, false>, grid, block, 0, s, true, (const float*)x, ldx, (const float*)w,
-                      stride, offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
+        e = mg_launch(few ? narrow[form] : wide[form], tgrid, dim3(128), few ? moe_mma_smem(64, 4) : moe_mma_smem(128, 2), s, true,
+                      (const bf16*)x, ldx, (const bf16*)w, stride, offsets, slot_entry, top, scale, out, N, K, x_rows, act, limit);
+    } else if (is_bf16) {
+        auto kernel = form == 1 ? moe_gemm_kernel<bf16, 1> : form == 2 ? moe_gemm_kernel<bf16, 2> : moe_gemm_kernel<bf16, 0>;
+        e = mg_launch(kernel, grid, block, 0, s, true, (const bf16*)x, ldx, (const bf16*)w, stride, offsets, slot_entry, top, scale,
+                      out, N, K, x_rows, act, limit);
+    } else {
+        auto kernel = form == 1 ? moe_gemm_kernel<float, 1> : form == 2 ? moe_gemm_kernel<float, 2> : moe_gemm_kernel<float, 0>;
+        e = mg_launch(kernel, grid, block, 0, s, true, (const float*)x, ldx, (const float*)w, stride, offsets, slot_entry, top,
+                      scale, out, N, K, x_rows, act, limit);
+    }
     MG_LAUNCHED(e, "moe gemm");
     return MG_OK;
 }

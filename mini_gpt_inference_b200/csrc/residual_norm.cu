@@ -1,9 +1,12 @@
 // What a layer with a norm on both sides of each sublayer, a loop over layers with an additive re-entry, and a
 // per-layer token input add to the 32-bit residual stream; all sums and statistics 32-bit.
 //
-// rmsnorm_add:  x += (y / sqrt(mean(y^2) + eps)) * (offset + w),  y = sa * a [+ sb * b]   (one warp a row; the
-//               sublayer's output a, or the weighted sum of two sublayers that ran side by side).  With `clear` the
-//               inputs are left as zeros: the buffer a sublayer added its output into serves the next sublayer as it is
+// norm_add:     x += scale * (y / sqrt(mean(y^2) + eps)) * (offset + w),  y = sa * a [+ sb * b]  (the sublayer's output a,
+//               or the weighted sum of two sublayers that ran side by side), or the sum of the rows that a token's
+//               entries point to (experts that wrote their results apart); with `center` the mean of y is taken off
+//               first (a layer norm).  With `clear` the inputs are left as zeros: the buffer a sublayer added its output
+//               into serves the next sublayer as it is.  Optionally the new x is also written in bfloat16: what a
+//               sublayer that reads the stream itself wants next
 // add_rows:     x += [e] + v    (e: rows like x, or none; v: one row for all tokens)
 // scaled_sum:   x += sa * a + sb * b   (with `clear`, a and b are left as zeros)
 // softcap:      x <- cap * tanh(x / cap)
@@ -22,81 +25,161 @@ constexpr int NORM_WARPS = 4;
 constexpr int ROW_THREADS = 256;   // threads of the CTA that owns a row in the vector form
 constexpr int MAX_ROW_VECS = 8;    // most float4 a thread holds: rows of up to 256 * 8 * 4 = 8,192 numbers
 
-// The general form: one warp a row, two passes over the row (any width).
+// What the norm behind a sublayer reads: y = sa * a [+ sb * b], or, with `entry_slot`, the sum over a row's `top` entries
+// of the rows of `a` that they point to (entries below zero: none), in entry order.
+struct NormInput {
+    float* a;
+    float sa;
+    float* b;
+    float sb;
+    const int* entry_slot;         // [rows, top] or null
+    int top, n_slots;
+};
+
+struct NormOutput {
+    float* x;                      // the stream, in place
+    const float* w;
+    float eps, offset, scale;      // x += scale * norm(y) * (offset + w)
+    int center;                    // take the row's mean off first (a layer norm)
+    int clear;                     // leave a and b as zeros
+    bf16* rows;                    // the new stream in bfloat16 as well, or null
+};
+
+__device__ __forceinline__ int entry_row(const NormInput& in, size_t row, int k) {
+    const int slot = in.entry_slot[row * in.top + k];
+    return slot >= 0 && MG_GUARDED(residual_norm, MG_GUARD_ROW, slot, in.n_slots) ? slot : -1;
+}
+
+__device__ __forceinline__ float norm_input(const NormInput& in, size_t row, int width, int c) {
+    if (in.entry_slot == nullptr) {
+        const size_t i = row * width + c;
+        return in.b ? fmaf(in.sb, in.b[i], in.sa * in.a[i]) : in.sa * in.a[i];
+    }
+    float sum = 0.f;
+    for (int k = 0; k < in.top; ++k) {
+        const int slot = entry_row(in, row, k);
+        if (slot >= 0) sum += in.a[(size_t)slot * width + c];
+    }
+    return sum;
+}
+
+// The general form: one warp a row, two or three passes over the row (any width).
 __global__ void __launch_bounds__(32 * NORM_WARPS)
-rmsnorm_add_kernel(float* __restrict__ x, float* __restrict__ a, float sa, float* __restrict__ b, float sb,
-                   const float* __restrict__ w, int rows, int width, float eps, float offset, int clear) {
+norm_add_kernel(const NormInput in, const NormOutput out, int rows, int width) {
     pdl_trigger();
     pdl_wait();
     const int row = blockIdx.x * NORM_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= rows) return;
-    float* ar = a + (size_t)row * width;
-    float* br = b ? b + (size_t)row * width : nullptr;
+    float mean = 0.f;
+    if (out.center) {
+        for (int c = lane; c < width; c += 32) mean += norm_input(in, row, width, c);
+        mean = warp_sum(mean) / (float)width;
+    }
     float sq = 0.f;
     for (int c = lane; c < width; c += 32) {
-        const float y = br ? fmaf(sb, br[c], sa * ar[c]) : sa * ar[c];
+        const float y = norm_input(in, row, width, c) - mean;
         sq = fmaf(y, y, sq);
     }
-    const float rstd = 1.0f / sqrtf(warp_sum(sq) / (float)width + eps);
-    float* xr = x + (size_t)row * width;
+    const float rstd = 1.0f / sqrtf(warp_sum(sq) / (float)width + out.eps);
     for (int c = lane; c < width; c += 32) {
-        const float y = br ? fmaf(sb, br[c], sa * ar[c]) : sa * ar[c];
-        xr[c] += y * rstd * (offset + w[c]);
-        if (clear) {
-            ar[c] = 0.f;
-            if (br) br[c] = 0.f;
+        const size_t i = (size_t)row * width + c;
+        const float y = norm_input(in, row, width, c) - mean;
+        const float x = out.x[i] + out.scale * (y * rstd * (out.offset + out.w[c]));
+        out.x[i] = x;
+        if (out.rows) out.rows[i] = __float2bfloat16_rn(x);
+        if (out.clear) {
+            in.a[i] = 0.f;
+            if (in.b) in.b[i] = 0.f;
         }
     }
+}
+
+__device__ __forceinline__ float row_total(float v, float* red) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int k = 0; k < ROW_THREADS / 32; ++k) total += red[k];
+    return total;
 }
 
 // The vector form: one CTA a row, the row's numbers asked for at once (16 bytes a load) and held in registers
 // between the statistics and the sum, so that a step of few rows is one trip to memory and not a chain of them.
 template <int ROW_VECS>       // float4 a thread holds: 1, 2, 4 or 8 (rows of up to 1,024 ... 8,192 numbers)
 __global__ void __launch_bounds__(ROW_THREADS)
-rmsnorm_add_vec_kernel(float* __restrict__ x, float* __restrict__ a, float sa, float* __restrict__ b, float sb,
-                       const float* __restrict__ w, int width, float eps, float offset, int clear) {
-    __shared__ float red[ROW_THREADS / 32];
+norm_add_vec_kernel(const NormInput in, const NormOutput out, int width) {
+    __shared__ float red[2][ROW_THREADS / 32];
     pdl_trigger();
     pdl_wait();
     const int vecs = width >> 2, tid = threadIdx.x;
-    float4* ar = reinterpret_cast<float4*>(a + (size_t)blockIdx.x * width);
-    float4* br = b ? reinterpret_cast<float4*>(b + (size_t)blockIdx.x * width) : nullptr;
-    float4* xr = reinterpret_cast<float4*>(x + (size_t)blockIdx.x * width);
-    const float4* wr = reinterpret_cast<const float4*>(w);
+    const size_t row = blockIdx.x, base = row * vecs;
+    float4* ar = reinterpret_cast<float4*>(in.a) + base;
+    float4* br = in.b ? reinterpret_cast<float4*>(in.b) + base : nullptr;
+    float4* xr = reinterpret_cast<float4*>(out.x) + base;
+    const float4* wr = reinterpret_cast<const float4*>(out.w);
     float4 y[ROW_VECS], xv[ROW_VECS], wv[ROW_VECS];
 #pragma unroll
     for (int u = 0; u < ROW_VECS; ++u) {
         const int i = tid + u * ROW_THREADS;
         y[u] = xv[u] = wv[u] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (i < vecs) {
-            const float4 av = ar[i];
-            y[u] = make_float4(sa * av.x, sa * av.y, sa * av.z, sa * av.w);
-            if (br) {
-                const float4 bv = br[i];
-                y[u] = make_float4(fmaf(sb, bv.x, y[u].x), fmaf(sb, bv.y, y[u].y), fmaf(sb, bv.z, y[u].z), fmaf(sb, bv.w, y[u].w));
+            if (in.entry_slot == nullptr) {
+                const float4 av = ar[i];
+                y[u] = make_float4(in.sa * av.x, in.sa * av.y, in.sa * av.z, in.sa * av.w);
+                if (br) {
+                    const float4 bv = br[i];
+                    y[u] = make_float4(fmaf(in.sb, bv.x, y[u].x), fmaf(in.sb, bv.y, y[u].y), fmaf(in.sb, bv.z, y[u].z), fmaf(in.sb, bv.w, y[u].w));
+                }
             }
             xv[u] = xr[i];
             wv[u] = wr[i];
         }
     }
+    if (in.entry_slot != nullptr) {
+#pragma unroll 4
+        for (int k = 0; k < in.top; ++k) {
+            const int slot = entry_row(in, row, k);
+            if (slot < 0) continue;
+            const float4* tr = reinterpret_cast<const float4*>(in.a) + (size_t)slot * vecs;
+#pragma unroll
+            for (int u = 0; u < ROW_VECS; ++u) {
+                const int i = tid + u * ROW_THREADS;
+                if (i < vecs) {
+                    const float4 av = tr[i];
+                    y[u] = make_float4(y[u].x + av.x, y[u].y + av.y, y[u].z + av.z, y[u].w + av.w);
+                }
+            }
+        }
+    }
+    if (out.center) {
+        float sum = 0.f;
+#pragma unroll
+        for (int u = 0; u < ROW_VECS; ++u) sum += (y[u].x + y[u].y) + (y[u].z + y[u].w);
+        const float mean = row_total(sum, red[0]) / (float)width;
+#pragma unroll
+        for (int u = 0; u < ROW_VECS; ++u)
+            if (tid + u * ROW_THREADS < vecs) y[u] = make_float4(y[u].x - mean, y[u].y - mean, y[u].z - mean, y[u].w - mean);
+    }
     float sq = 0.f;
 #pragma unroll
     for (int u = 0; u < ROW_VECS; ++u) sq = fmaf(y[u].x, y[u].x, fmaf(y[u].y, y[u].y, fmaf(y[u].z, y[u].z, fmaf(y[u].w, y[u].w, sq))));
-    sq = warp_sum(sq);
-    if ((tid & 31) == 0) red[tid >> 5] = sq;
-    __syncthreads();
-    float total = 0.f;
-#pragma unroll
-    for (int k = 0; k < ROW_THREADS / 32; ++k) total += red[k];
-    const float rstd = 1.0f / sqrtf(total / (float)width + eps);
+    const float rstd = 1.0f / sqrtf(row_total(sq, red[1]) / (float)width + out.eps);
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float sc = out.scale, off = out.offset;
 #pragma unroll
     for (int u = 0; u < ROW_VECS; ++u) {
         const int i = tid + u * ROW_THREADS;
         if (i < vecs) {
-            xr[i] = make_float4(xv[u].x + y[u].x * rstd * (offset + wv[u].x), xv[u].y + y[u].y * rstd * (offset + wv[u].y),
-                                xv[u].z + y[u].z * rstd * (offset + wv[u].z), xv[u].w + y[u].w * rstd * (offset + wv[u].w));
-            if (clear) {
+            const float4 r = make_float4(xv[u].x + sc * (y[u].x * rstd * (off + wv[u].x)), xv[u].y + sc * (y[u].y * rstd * (off + wv[u].y)),
+                                         xv[u].z + sc * (y[u].z * rstd * (off + wv[u].z)), xv[u].w + sc * (y[u].w * rstd * (off + wv[u].w)));
+            xr[i] = r;
+            if (out.rows) {
+                __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(out.rows + 4 * (base + i));
+                o[0] = __floats2bfloat162_rn(r.x, r.y);
+                o[1] = __floats2bfloat162_rn(r.z, r.w);
+            }
+            if (out.clear) {
                 ar[i] = zero;
                 if (br) br[i] = zero;
             }
@@ -171,21 +254,28 @@ __global__ void token_gate_kernel(const float* __restrict__ g, const int* __rest
 }  // namespace
 
 // x: [rows, width] 32-bit, in place; a (and b, or null): [rows, width] 32-bit (zeroed if clear); w: [width] 32-bit.
-MG_API int mg_rmsnorm_add(float* x, float* a, float sa, float* b, float sb, const float* w, int rows,
-                          int width, float eps, float offset, int clear, void* stream) {
+// center: the row's mean is taken off first.  scale: factor on what is added.  out_rows: [rows, width] bfloat16 or null.
+// entry_slot (or null): [rows, top] rows of a, [n_slots, width], whose sum is the input (below zero: none); then b must be
+// null and clear 0.
+MG_API int mg_norm_add(float* x, float* a, float sa, float* b, float sb, const int* entry_slot, int top, int n_slots,
+                       const float* w, int rows, int width, float eps, float offset, int center, float scale, int clear,
+                       void* out_rows, void* stream) {
     if (rows == 0) return MG_OK;
-    MG_REQUIRE(rows > 0 && width > 0 && x && a && w, "rmsnorm_add: bad sizes");
+    MG_REQUIRE(rows > 0 && width > 0 && x && a && w, "norm_add: bad sizes");
+    MG_REQUIRE(entry_slot == nullptr || (top > 0 && n_slots > 0 && b == nullptr && !clear && sa == 1.f),
+               "norm_add: a sum over entries takes neither a second input nor a factor, and is not cleared");
+    const NormInput in{a, sa, b, sb, entry_slot, top, n_slots};
+    const NormOutput out{x, w, eps, offset, scale, center, clear, (bf16*)out_rows};
     const bool vec = width % 4 == 0 && width <= ROW_THREADS * MAX_ROW_VECS * 4 && (uintptr_t)x % 16 == 0 && (uintptr_t)a % 16 == 0 &&
-                     (uintptr_t)b % 16 == 0 && (uintptr_t)w % 16 == 0;
+                     (uintptr_t)b % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out_rows % 4 == 0;
     const int per_thread = ceil_div(width / 4, ROW_THREADS);
-    auto vec_kernel = per_thread <= 1 ? rmsnorm_add_vec_kernel<1> : per_thread <= 2 ? rmsnorm_add_vec_kernel<2>
-                    : per_thread <= 4 ? rmsnorm_add_vec_kernel<4> : rmsnorm_add_vec_kernel<8>;
+    auto vec_kernel = per_thread <= 1 ? norm_add_vec_kernel<1> : per_thread <= 2 ? norm_add_vec_kernel<2>
+                    : per_thread <= 4 ? norm_add_vec_kernel<4> : norm_add_vec_kernel<8>;
     const cudaError_t e =
-        vec ? mg_launch(vec_kernel, dim3(rows), dim3(ROW_THREADS), 0, (cudaStream_t)stream, true, x, a, sa, b, sb, w,
-                        width, eps, offset, clear)
-            : mg_launch(rmsnorm_add_kernel, dim3(ceil_div(rows, NORM_WARPS)), dim3(32 * NORM_WARPS), 0, (cudaStream_t)stream,
-                        true, x, a, sa, b, sb, w, rows, width, eps, offset, clear);
-    if (e != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "rmsnorm_add: %s", cudaGetErrorString(e));
+        vec ? mg_launch(vec_kernel, dim3(rows), dim3(ROW_THREADS), 0, (cudaStream_t)stream, true, in, out, width)
+            : mg_launch(norm_add_kernel, dim3(ceil_div(rows, NORM_WARPS)), dim3(32 * NORM_WARPS), 0, (cudaStream_t)stream,
+                        true, in, out, rows, width);
+    if (e != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "norm_add: %s", cudaGetErrorString(e));
     return MG_OK;
 }
 

@@ -18,7 +18,8 @@
 // made from one small latent per token:
 //   * the first C numbers of `low`, RMS-normed with a gain, are the latent; the last R turn with the position
 //     and are one key part that all heads share; [latent | turned part] is the token's one cache row (and the
-//     latent alone its value row, where values have pages of their own);
+//     latent alone its value row, where values have pages of their own); features d and d + R/2 turn together, or
+//     neighbours 2i and 2i + 1, cosine and sine times a factor (stretched frequencies come with one);
 //   * the last R features of every query head turn the same way and are written to a second tensor, behind the
 //     C numbers per head that a per-head product fills in: rows [H x (C + R)].
 //
@@ -171,12 +172,20 @@ rotate_heads_kernel(T* __restrict__ x, int n_head, int v_dim, const float* __res
     }
 }
 
+// Which pair a turning feature belongs to, its partner, and whether it is the pair's first: features d and d + R/2, or
+// (neighbours) 2i and 2i + 1.
+struct TurnPair { int pair, partner; bool first; };
+__device__ __forceinline__ TurnPair turn_pair(int d, int half, int neighbours) {
+    if (neighbours) return {d >> 1, d ^ 1, (d & 1) == 0};
+    return d < half ? TurnPair{d, d + half, true} : TurnPair{d - half, d - half, false};
+}
+
 template <typename T>
 __global__ void __launch_bounds__(THREADS)
 latent_prepare_kernel(const T* __restrict__ proj, int ld, int n_head, int q_off, int q_dim, int rot, int low_off, int rank,
                       const float* __restrict__ gain, float eps, const float* __restrict__ freq, T* __restrict__ q_out,
                       const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ k_pages,
-                      T* __restrict__ v_pages, int page_tokens, int num_pages) {
+                      T* __restrict__ v_pages, int page_tokens, int num_pages, int neighbours, float magnitude) {
     extern __shared__ float smem[];                        // [rank + rot] low, [rot] cos/sin pairs
     __shared__ float red[THREADS / 32];
     pdl_trigger();
@@ -192,8 +201,8 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, int n_head, int q_off,
         const float a = __fmul_rn((float)pos, freq[i]);
         float s, c;
         sincosf(a, &s, &c);
-        cs[2 * i] = c;
-        cs[2 * i + 1] = s;
+        cs[2 * i] = c * magnitude;
+        cs[2 * i + 1] = s * magnitude;
     }
     int slot = slots ? slots[token] : -1;
     if (slot >= 0 && !MG_GUARDED(rotary_prepare, MG_GUARD_CACHE_ROW, slot, (long long)num_pages * page_tokens)) slot = -1;
@@ -212,10 +221,10 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, int n_head, int q_off,
     for (int i = tid; i < n_head * rot; i += THREADS) {
         const int h = i / rot, d = i - h * rot;
         const T* qh = row + q_off + (size_t)h * (q_dim + rot) + q_dim;
-        const int j = d < half ? d : d - half;
-        const float x = to_float(qh[d]), y = to_float(qh[d < half ? d + half : d - half]);
-        const float c = cs[2 * j], s = cs[2 * j + 1];
-        q_out[((size_t)token * n_head + h) * out_head + rank + d] = from_float<T>(d < half ? x * c - y * s : x * c + y * s);
+        const TurnPair p = turn_pair(d, half, neighbours);
+        const float x = to_float(qh[d]), y = to_float(qh[p.partner]);
+        const float c = cs[2 * p.pair], s = p.first ? -cs[2 * p.pair + 1] : cs[2 * p.pair + 1];
+        q_out[((size_t)token * n_head + h) * out_head + rank + d] = from_float<T>(x * c + y * s);
     }
     if (!store) return;
     const float r = 1.0f / sqrtf(total / (float)rank + eps);
@@ -228,10 +237,10 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, int n_head, int q_off,
         if (vrow) vrow[i] = c;
     }
     for (int d = tid; d < rot; d += THREADS) {
-        const int j = d < half ? d : d - half;
-        const float x = low[rank + d], y = low[rank + (d < half ? d + half : d - half)];
-        const float c = cs[2 * j], s = cs[2 * j + 1];
-        krow[rank + d] = from_float<T>(d < half ? x * c - y * s : x * c + y * s);
+        const TurnPair p = turn_pair(d, half, neighbours);
+        const float x = low[rank + d], y = low[rank + p.partner];
+        const float c = cs[2 * p.pair], s = p.first ? -cs[2 * p.pair + 1] : cs[2 * p.pair + 1];
+        krow[rank + d] = from_float<T>(x * c + y * s);
     }
 }
 
@@ -298,11 +307,11 @@ MG_API int mg_rotate_heads(void* x, int n_tokens, int n_head, int v_dim, const f
 // latents of its own (k_pages not null), `low` (rank + rot numbers from low_off); gain: [rank] 32-bit; freq:
 // [rot / 2]; q_out: [n_tokens, n_head * (rank + rot)], of which the last rot of every head are written; key pages
 // [page, 1, page_tokens, rank + rot]; value pages [page, 1, page_tokens, rank] or null (values read from the key
-// rows).
+// rows).  neighbours: features 2i and 2i + 1 turn together (else i and i + rot / 2); magnitude: factor on cosine and sine.
 MG_API int mg_latent_prepare(const void* proj, int ld, int n_tokens, int n_head, int q_off, int q_dim, int rot, int low_off,
                              int rank, const float* gain, float eps, const float* freq, void* q_out, const int* positions,
                              const int* slots, void* k_pages, void* v_pages, int page_tokens, int num_pages, int is_bf16,
-                             void* stream) {
+                             int neighbours, float magnitude, void* stream) {
     if (n_tokens == 0) return MG_OK;
     MG_REQUIRE(n_tokens > 0 && n_head > 0 && q_dim > 0 && rank > 0 && positions != nullptr && q_out != nullptr,
                "latent_prepare: bad sizes");
@@ -320,13 +329,13 @@ MG_API int mg_latent_prepare(const void* proj, int ld, int n_tokens, int n_head,
         if (e == cudaSuccess)
             e = mg_launch(latent_prepare_kernel<bf16>, dim3(n_tokens), dim3(THREADS), smem, s, true, (const bf16*)proj, ld,
                           n_head, q_off, q_dim, rot, low_off, rank, gain, eps, freq, (bf16*)q_out, positions, slots,
-                          (bf16*)k_pages, (bf16*)v_pages, page_tokens, num_pages);
+                          (bf16*)k_pages, (bf16*)v_pages, page_tokens, num_pages, neighbours, magnitude);
     } else {
         e = smem > 48 * 1024 ? cudaFuncSetAttribute(latent_prepare_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) : cudaSuccess;
         if (e == cudaSuccess)
             e = mg_launch(latent_prepare_kernel<float>, dim3(n_tokens), dim3(THREADS), smem, s, true, (const float*)proj, ld,
                           n_head, q_off, q_dim, rot, low_off, rank, gain, eps, freq, (float*)q_out, positions, slots,
-                          (float*)k_pages, (float*)v_pages, page_tokens, num_pages);
+                          (float*)k_pages, (float*)v_pages, page_tokens, num_pages, neighbours, magnitude);
     }
     if (e != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "latent_prepare: %s", cudaGetErrorString(e));
     return MG_OK;

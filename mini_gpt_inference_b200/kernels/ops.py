@@ -18,6 +18,7 @@ from .attention_plan import KEY_CHUNK, query_tiles
 from .library import KernelLibraryError, check
 
 EPILOGUES = {"none": 0, "gelu_tanh": 1, "residual": 2, "relu_sq": 3}
+PLAIN_ACTIVATIONS = {"relu_sq": 0, "gelu_tanh": 1, "silu": 2}           # ... and the activation of a unit without a gate
 GATED_ACTIVATIONS = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 2}     # the gated product of a unit's two halves
 SKINNY_ROWS = 16         # most tokens the small-batch projection kernel takes
 CLUSTER_ROWS = 128       # most tokens the mid-batch (K split over a cluster) projection kernel takes
@@ -59,6 +60,15 @@ class DeferredRMSNorm(DeferredNorm):
     def _materialize(self):
         x = self.x32 if self.rows is None else self.ops.gather_rows(self.x32, self.rows)
         return self.ops.rmsnorm(x, self.weight, -self.eps, self.offset, self.dtype)
+
+
+class EntrySum:
+    """Per-token sums that have not been taken yet: row ``t`` is the sum of the rows of ``terms`` that ``entry_slot[t]``
+    points to (below zero: none).  The norm behind a sublayer takes the sum on its way (``norm_add``)."""
+
+    def __init__(self, terms, entry_slot) -> None:
+        self.terms, self.entry_slot = terms, entry_slot
+        self.shape = (entry_slot.shape[0], terms.shape[1])
 
 
 _raw_stream = getattr(torch._C, "_cuda_getCurrentRawStream", None)
@@ -968,11 +978,7 @@ class CudaOps:
             group = n_head // n_kv_head
             args = None
             if single:
-                keys = self.lib.mg_attention_mma_split_keys(int(ctx.max_ctx_after))
-                # (with a block mask a token's keys begin at its block: ranges are counted from the key
-                # block of 64 that holds the block's first position)
-                span = int(ctx.max_ctx_after) if block <= 0 else min(int(ctx.max_ctx_after), block + 64)
-                splits = max(1, -(-span // keys))
+                keys, splits = self._key_ranges(int(ctx.max_ctx_after), int(cache.window or 0), block)
                 floats = self.lib.mg_attention_mma_scratch_floats(n, n_head, v_dim, splits)
                 scratch = torch.empty((floats,), dtype=torch.float32, device=self.device)
                 # (measured at batch 8, context 2,048: the ranges merged by a second kernel, 0.273 ms a
@@ -1003,8 +1009,7 @@ class CudaOps:
             group = n_head // n_kv_head
             args = None
             if single:
-                keys = self.lib.mg_attention_mma_split_keys(int(ctx.max_ctx_after))
-                splits = max(1, -(-int(ctx.max_ctx_after) // keys))
+                keys, splits = self._key_ranges(int(ctx.max_ctx_after), int(cache.window or 0), 0)
                 floats = self.lib.mg_attention_mma_scratch_floats(n, n_head, v_dim, splits)
                 scratch = torch.empty((floats,), dtype=torch.float32, device=self.device)
                 args = [_ptr(scratch), 1, 0, splits, keys]
@@ -1029,6 +1034,17 @@ class CudaOps:
             float(scale), cache.k_pages.shape[0], table.shape[0], self._is_bf16(q), _ptr(slopes), block,
             softcap, _ptr(sinks), head_dim if in_keys else 0, self._stream()), "paged_attention (general)")
         return out
+
+    def _key_ranges(self, max_context, window, block):
+        """Keys per range and ranges per token for single tokens with contexts of up to ``max_context`` keys.  With a
+        window or a block mask a token's keys begin at its own first position: ranges are counted from the key block of
+        64 that holds it, so they cover at most the window's (the block's) length and 63 keys in front of it."""
+        span = max_context
+        for reach in (window, block):
+            if reach > 0:
+                span = min(span, reach + 64)
+        keys = self.lib.mg_attention_mma_split_keys(span)
+        return keys, max(1, -(-span // keys))
 
     # ---- several residual streams ------------------------------------------------------------------
     def streams_spread(self, x32, streams):
@@ -1179,19 +1195,43 @@ class CudaOps:
             shared[key] = out
         return out
 
-    def rmsnorm_add(self, residual32, y32, weight, eps, offset=0.0, other32=None, scale=1.0, other_scale=1.0, clear=False):
-        """``residual32 += rms_norm(scale * y32 [+ other_scale * other32]) * (offset + weight)``, in place, 32-bit.
-        ``clear``: ``y32`` (and ``other32``) are left as zeros, ready for the next sublayer to add into."""
+    def norm_add(self, residual32, y32, weight, eps, offset=0.0, center=False, norm_scale=1.0, other32=None, scale=1.0,
+                 other_scale=1.0, clear=False, rows_dtype=None):
+        """``residual32 += norm_scale * norm(scale * y32 [+ other_scale * other32]) * (offset + weight)``, in place, 32-bit:
+        an RMS norm, or with ``center`` a layer norm without a shift.  ``y32`` may be an ``EntrySum``: the norm then takes
+        the sum on its way.  ``clear``: ``y32`` (and ``other32``) are left as zeros, ready for the next sublayer to add
+        into.  With ``rows_dtype`` the new stream is also returned in that type (``residual32`` itself if 32-bit)."""
         self._want(residual32, torch.float32, "residual", 2)
-        self._want(y32, torch.float32, "sublayer output", 2)
+        entries = [None, 0, 0]
+        terms = y32
+        if isinstance(y32, EntrySum):
+            terms = y32.terms
+            self._want(y32.entry_slot, torch.int32, "entry slots", 2)
+            if other32 is not None or clear or scale != 1.0:
+                raise KernelLibraryError("norm_add: a sum over entries takes neither a second input nor a factor")
+            entries = [_ptr(y32.entry_slot), y32.entry_slot.shape[1], terms.shape[0]]
+        self._want(terms, torch.float32, "sublayer output", 2)
         self._want(weight, torch.float32, "norm weight", 1)
         if other32 is not None:
             self._want(other32, torch.float32, "second sublayer output", 2)
-        if y32.shape != residual32.shape or weight.numel() != residual32.shape[1] or (other32 is not None and other32.shape != y32.shape):
-            raise KernelLibraryError("rmsnorm_add: shapes do not fit")
-        self._run(self.lib.mg_rmsnorm_add(_ptr(residual32), _ptr(y32), float(scale), _ptr(other32), float(other_scale),
-                                          _ptr(weight), residual32.shape[0], residual32.shape[1], float(eps), float(offset),
-                                          1 if clear else 0, self._stream()), "rmsnorm_add")
+        if (tuple(y32.shape) != tuple(residual32.shape) or weight.numel() != residual32.shape[1]
+                or (other32 is not None and other32.shape != y32.shape)):
+            raise KernelLibraryError("norm_add: shapes do not fit")
+        rows = residual32 if rows_dtype == torch.float32 else None
+        if rows_dtype == torch.bfloat16:
+            rows = torch.empty(residual32.shape, dtype=rows_dtype, device=self.device)
+        elif rows_dtype not in (None, torch.float32):
+            raise KernelLibraryError(f"norm_add: rows in {rows_dtype}")
+        self._run(self.lib.mg_norm_add(
+            _ptr(residual32), _ptr(terms), float(scale), _ptr(other32), float(other_scale), *entries, _ptr(weight),
+            residual32.shape[0], residual32.shape[1], float(eps), float(offset), 1 if center else 0, float(norm_scale),
+            1 if clear else 0, _ptr(rows) if rows_dtype == torch.bfloat16 else None, self._stream()), "norm_add")
+        return rows
+
+    def rmsnorm_add(self, residual32, y32, weight, eps, offset=0.0, other32=None, scale=1.0, other_scale=1.0, clear=False):
+        """``residual32 += rms_norm(scale * y32 [+ other_scale * other32]) * (offset + weight)``, in place, 32-bit.
+        ``clear``: ``y32`` (and ``other32``) are left as zeros, ready for the next sublayer to add into."""
+        self.norm_add(residual32, y32, weight, eps, offset, other32=other32, scale=scale, other_scale=other_scale, clear=clear)
         return residual32
 
     def add_rows(self, x32, rows32, vector):
@@ -1273,12 +1313,14 @@ class CudaOps:
                                          self._is_bf16(table), self._is_bf16(out), self._stream()), "token_gate")
         return out
 
-    def latent_prepare(self, proj, n_head, q_off, q_dim, rot_dim, low_off, rank, gain, eps, freq, cache, slots, positions):
+    def latent_prepare(self, proj, n_head, q_off, q_dim, rot_dim, low_off, rank, gain, eps, freq, cache, slots, positions,
+                       neighbours=False, magnitude=1.0):
         """For an attention over cached latents.  Returns ``q`` ``[tokens, n_head * (rank + rot_dim)]`` whose last
         ``rot_dim`` features per head are the turned last ``rot_dim`` features of the query heads in ``proj``
         (``n_head x (q_dim + rot_dim)`` from ``q_off``); the first ``rank`` per head are left for ``head_linear``.
         With a writable ``cache``: the ``rank`` numbers of ``proj`` from ``low_off``, RMS-normed with ``gain``, and the
-        ``rot_dim`` behind them, turned, go to the token's cache row."""
+        ``rot_dim`` behind them, turned, go to the token's cache row.  Feature ``i`` of a turning part pairs with ``i +
+        rot_dim / 2``, or, with ``neighbours``, ``2i`` with ``2i + 1``; ``magnitude``: factor on cosine and sine."""
         self._want(proj, None, "projection rows", 2)
         self._want(positions, torch.int32, "positions", 1)
         if rot_dim and self._want(freq, torch.float32, "rotary frequencies", 1).numel() != rot_dim // 2:
@@ -1298,7 +1340,7 @@ class CudaOps:
         self._run(self.lib.mg_latent_prepare(
             _ptr(proj), proj.shape[1], proj.shape[0], n_head, q_off, q_dim, int(rot_dim), low_off, rank, _ptr(gain),
             float(eps), _ptr(freq), _ptr(q), _ptr(positions), pages[0], pages[1], pages[2], pages[3], pages[4],
-            self._is_bf16(proj), self._stream()), "latent_prepare")
+            self._is_bf16(proj), 1 if neighbours else 0, float(magnitude), self._stream()), "latent_prepare")
         return q
 
     def head_linear(self, x, x_off, x_head, weight, rows_are_inputs, n_head, n_in, n_out, gate=None, out=None, out_off=0,
@@ -1372,26 +1414,29 @@ class CudaOps:
         return out
 
     # ---- routed experts ---------------------------------------------------------------------------
-    def moe_route(self, y, router_weight, gate_weight, positions, top):
+    def moe_route(self, y, router_weight, gate_weight, positions, top, always=0):
         """Router of a feed-forward of experts: returns (ids [tokens, top] int32, weights [tokens,
         top] 32-bit, gate [tokens] 32-bit or None): the ``top`` largest of ``router_weight @ y``
-        with the softmax over them, and the logistic function of ``gate_weight . y``."""
+        with the softmax over them, and the logistic function of ``gate_weight . y``.  ``always`` experts behind the
+        router's own (numbers ``experts ..``) join every token's chosen ones as further columns of ids and weights, with
+        the gate's value (1 without one) as their weight; then no gate is returned."""
         self._want(y, None, "router input", 2)
         self._want(router_weight, torch.float32, "router weight", 2)
         n, width = y.shape
         experts = router_weight.shape[0]
-        if router_weight.shape[1] != width or not 0 < top <= experts:
+        if router_weight.shape[1] != width or not 0 < top <= experts or always < 0:
             raise KernelLibraryError("moe_route: shapes do not fit")
-        ids = torch.empty((n, top), dtype=torch.int32, device=self.device)
-        weights = torch.empty((n, top), dtype=torch.float32, device=self.device)
+        ids = torch.empty((n, top + always), dtype=torch.int32, device=self.device)
+        weights = torch.empty((n, top + always), dtype=torch.float32, device=self.device)
         gate = None
         if gate_weight is not None:
             self._want(gate_weight, torch.float32, "gate weight")
             if gate_weight.numel() != width:
                 raise KernelLibraryError("moe_route: the gate's weights do not fit the width")
-            gate = torch.empty((n,), dtype=torch.float32, device=self.device)
+            if not always:
+                gate = torch.empty((n,), dtype=torch.float32, device=self.device)
         self._run(self.lib.mg_moe_route(_ptr(y), _ptr(router_weight), _ptr(gate_weight), _ptr(positions), _ptr(ids),
-                                        _ptr(weights), _ptr(gate), n, width, experts, top, self._is_bf16(y),
+                                        _ptr(weights), _ptr(gate), n, width, experts, top, int(always), self._is_bf16(y),
                                         self._stream()), "moe route")
         return ids, weights, gate
 
@@ -1426,39 +1471,47 @@ class CudaOps:
                                                self._is_bf16(y), self._stream()), "moe route (scored)")
         return ids, weights, gate
 
-    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0):
-        """``residual32[t] += sum_k weights[t, k] * expert(ids[t, k])(y[t])`` with expert e as
-        ``w_out[e] @ (silu(w_in[e][:F] @ y) * (w_in[e][F:] @ y))``; ``w_in`` [E, 2F, C], ``w_out``
-        [E, C, F].  Tokens are grouped by expert on the device; the host never learns the counts."""
+    def moe_experts(self, y, ids, weights, w_in, w_out, activation="silu", limit=0.0, gated=True):
+        """``sum_k weights[t, k] * expert(ids[t, k])(y[t])`` as an ``EntrySum`` (every entry's product apart), with expert
+        e as ``w_out[e] @ (silu(w_in[e][:F] @ y) * (w_in[e][F:] @ y))``, ``w_in`` [E, 2F, C], ``w_out`` [E, C, F], or, not
+        ``gated``, ``w_out[e] @ act(w_in[e] @ y)`` with ``w_in`` [E, F, C] (``activation``: ``relu_sq``, ``gelu_tanh``,
+        ``silu``).  Tokens are grouped by expert on the device; the host never learns the counts."""
         self._want(y, w_in.dtype, "expert input", 2)
         self._want(w_in, None, "expert matrices (in)", 3)
         self._want(w_out, w_in.dtype, "expert matrices (out)", 3)
-        self._want(residual32, torch.float32, "residual", 2)
         n, width = y.shape
-        experts, two_f, _ = w_in.shape
-        inner, top = two_f // 2, ids.shape[1]
-        if (w_in.shape != (experts, 2 * inner, width) or w_out.shape != (experts, width, inner)
-                or ids.shape[0] != n or weights.shape != ids.shape or residual32.shape != (n, width)):
+        experts, inner, top = w_in.shape[0], w_out.shape[2], ids.shape[1]
+        if (w_in.shape != (experts, (2 if gated else 1) * inner, width) or w_out.shape != (experts, width, inner)
+                or ids.shape[0] != n or weights.shape != ids.shape):
             raise KernelLibraryError("moe_experts: shapes do not fit")
         entries = n * top
         is_bf16 = self._is_bf16(y)
-        act = GATED_ACTIVATIONS[activation]
+        act = (GATED_ACTIVATIONS if gated else PLAIN_ACTIVATIONS)[activation]
         offsets = torch.empty((experts + 1,), dtype=torch.int32, device=self.device)
         slot_entry = torch.empty((entries,), dtype=torch.int32, device=self.device)
-        entry_slot = torch.empty((entries,), dtype=torch.int32, device=self.device)
+        entry_slot = torch.empty((n, top), dtype=torch.int32, device=self.device)
         self._run(self.lib.mg_moe_group(_ptr(ids), entries, experts, _ptr(offsets), _ptr(slot_entry), _ptr(entry_slot),
                                         self._stream()), "moe group")
         hidden = torch.empty((entries, inner), dtype=y.dtype, device=self.device)
         self._run(self.lib.mg_moe_gemm(_ptr(y), width, _ptr(w_in), _ptr(offsets), _ptr(slot_entry), top, None,
-                                       _ptr(hidden), experts, n, inner, width, n, 1, is_bf16, act, float(limit),
+                                       _ptr(hidden), experts, n, inner, width, n, 1 if gated else 2, is_bf16, act, float(limit),
                                        self._stream()),
                   "moe experts (in)")
         out = torch.empty((entries, width), dtype=torch.float32, device=self.device)
         self._run(self.lib.mg_moe_gemm(_ptr(hidden), inner, _ptr(w_out), _ptr(offsets), _ptr(slot_entry), top,
                                        _ptr(weights), _ptr(out), experts, n, width, inner, entries, 0, is_bf16, 0, 0.0,
                                        self._stream()), "moe experts (out)")
-        self._run(self.lib.mg_moe_combine(_ptr(out), _ptr(entry_slot), top, _ptr(residual32), n, width, entries,
-                                          self._stream()), "moe combine")
+        return EntrySum(out, entry_slot)
+
+    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0, gated=True):
+        """``residual32[t] += `` the sum that ``moe_experts`` describes."""
+        self._want(residual32, torch.float32, "residual", 2)
+        if tuple(residual32.shape) != tuple(y.shape):
+            raise KernelLibraryError("moe_experts: the residual does not fit")
+        y = self.moe_experts(y, ids, weights, w_in, w_out, activation, limit, gated)
+        n, width = y.shape
+        self._run(self.lib.mg_moe_combine(_ptr(y.terms), _ptr(y.entry_slot), y.entry_slot.shape[1], _ptr(residual32), n, width,
+                                          y.terms.shape[0], self._stream()), "moe combine")
 
     def glu(self, gate_up, row_scale=None, activation="silu", limit=0.0):
         """``silu(gate_up[:, :F]) * gate_up[:, F:]``, each row times ``row_scale`` (32-bit ``[rows]``)

@@ -8,7 +8,8 @@ between a norm and the following projection is the compute dtype.
 
 Interfaces (what a new part must provide):
 
-* Norm:             ``forward(ctx, x32) -> y``            y in ctx.act_dtype, same shape
+* Norm:             ``forward(ctx, x32) -> y``            y in ctx.act_dtype, same shape; a norm that can stand behind
+                    a sublayer also has ``add_normed`` (reads the sublayer's output, adds into the stream)
 * PositionEncoding: ``table()`` (rows added to the token embedding, or None),
                     ``rotate(ctx, qkv, n_head, n_kv_head, head_dim)`` (in place on the q and
                     k columns of the fused projection; default no-op),
@@ -16,7 +17,9 @@ Interfaces (what a new part must provide):
 * Mixer:            built with ``position=`` (the model's position encoding),
                     ``cache_spec()`` (what the layer keeps per request, or None),
                     ``forward(ctx, cache, y, residual32)``  adds its output to residual32 in place
-                    and returns None, or returns another tensor that holds the sum
+                    and returns None, or returns another tensor that holds the sum; a part with
+                    ``returns_output`` also takes ``residual32=None`` and returns its output alone
+                    (32-bit rows, or an object that stands for them and that a norm can read)
 * FeedForward:      ``forward(ctx, y, residual32)``         the same
 * StreamEntry:      ``forward(ctx, x32, embedded32, index) -> x32``  a transformation of the whole residual
                     stream between layers (the re-entry of a loop over layers), given the embedding's output
@@ -33,6 +36,8 @@ from __future__ import annotations
 
 from typing import Any, Callable, Mapping
 
+import torch
+
 from .spec import PartSpec, TensorSpec
 
 
@@ -43,6 +48,9 @@ class Part:
     # True if forward() only launches kernels whose arguments do not change from step to step
     # (no host-side reads of the batch): such a part can be captured in a CUDA graph.
     graph_safe = False
+    # True if forward() takes residual32=None and then returns its output alone (an arrangement that
+    # does something with a sublayer's output before it joins the stream asks for that).
+    returns_output = False
 
     def __init__(self, prefix: str = "") -> None:
         self.prefix = prefix
@@ -63,6 +71,15 @@ class Part:
         for full_name in self.tensor_specs():
             local = full_name[len(self.prefix):].replace(".", "_")
             setattr(self, local, tensors.get(full_name))
+
+    @staticmethod
+    def add_output(ctx, rows, weight, residual32):
+        """A part's last projection: ``rows W^T`` added into ``residual32`` in place, or, without one, returned in
+        32-bit."""
+        if residual32 is None:
+            return ctx.ops.linear(rows, weight, None, "none", torch.float32)
+        ctx.ops.linear_residual(rows, weight, None, residual32)
+        return None
 
 
 class Norm(Part):

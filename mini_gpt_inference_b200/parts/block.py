@@ -13,6 +13,9 @@ returns the tensor that holds it at the end (or nothing, if that is the one it w
 feed-forward, ``x += norm2b(ff(norm2(x)))``, then, if it has one, the layer's token input (``side_input``), which
 reads the stream and the step's tokens and adds into the stream.  The sublayers add their output into a zeroed
 32-bit buffer; the norm behind them reads it and adds into the stream in one kernel.
+``post_norm``: norms behind the sublayers only, ``x += r * norm1(mixer(x))``, then, if the layer has a feed-forward,
+``x += r * norm2(ff(x))``, with ``r`` the layer's setting ``residual_scale``.  The sublayers read the stream itself, in the
+compute dtype; the norm behind a sublayer writes that copy of the new stream on its way, for the next sublayer or layer.
 """
 
 from __future__ import annotations
@@ -26,8 +29,9 @@ class Layer:
     """The built parts of one layer, by their names in the layer, and the arrangement's function."""
 
     def __init__(self, parts: dict[str, Any], roles: dict[str, str], run: Callable[..., None],
-                 prefix: str = "") -> None:
+                 prefix: str = "", settings: dict[str, Any] | None = None) -> None:
         self._parts = dict(parts)
+        self.settings = dict(settings or {})      # numbers of the arrangement itself
         self.roles = dict(roles)
         self.run = run
         self.prefix = prefix
@@ -109,3 +113,33 @@ def sandwich_norm(ctx, layer: Layer, cache, residual32):
 
 sandwich_norm.requires = ("norm1", "mixer", "norm1b")
 register_arrangement("sandwich_norm")(sandwich_norm)
+
+
+def _stream_rows(ctx, x):
+    """The stream in the compute dtype: the copy that the norm behind the last sublayer wrote, if it is of ``x``."""
+    kept = ctx.shared.get("stream rows")
+    return kept[1] if kept is not None and kept[0] is x else ctx.ops.cast(x, ctx.act_dtype)
+
+
+def post_norm(ctx, layer: Layer, cache, residual32):
+    x = residual32
+    r = layer.settings.get("residual_scale", 1.0)
+    rows = _stream_rows(ctx, x)
+
+    def add(part, norm, run):
+        if part.returns_output:
+            return norm.add_normed(ctx, run(None), x, scale=r, rows_dtype=ctx.act_dtype)
+        zeros = ctx.ops.zeros32(*x.shape, ctx)
+        y = stream_after(run(zeros), zeros)
+        return norm.add_normed(ctx, y, x, clear=y is zeros, scale=r, rows_dtype=ctx.act_dtype)
+    mixer, ff = layer.mixer, layer.get("feed_forward")
+    rows = add(mixer, layer.norm1, lambda into: mixer.forward(ctx, cache, rows, into))
+    if ff is not None:
+        rows = add(ff, layer.norm2, lambda into: ff.forward(ctx, rows, into))
+    ctx.shared["stream rows"] = (x, rows)
+    return None
+
+
+post_norm.requires = ("norm1", "mixer")
+post_norm.keeps_stream_rows = True     # leaves ctx.shared["stream rows"] valid for the layer that follows
+register_arrangement("post_norm")(post_norm)

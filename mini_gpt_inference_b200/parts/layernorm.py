@@ -40,6 +40,15 @@ class LayerNorm(Norm):
     def forward(self, ctx, x32):
         return ctx.ops.layernorm(x32, self.weight, self.bias, self.eps, ctx.act_dtype)
 
+    def add_normed(self, ctx, y32, residual32, clear=False, scale=1.0, rows_dtype=None):
+        """``residual32 += scale * norm(y32)`` in 32-bit, in place: the norm behind a sublayer (without a shift).
+        ``clear``: ``y32`` is left as zeros (a buffer that the next sublayer adds into).  With ``rows_dtype`` the new
+        stream is also returned in that type."""
+        if self.has_bias:
+            raise NotImplementedError("a norm behind a sublayer has no shift")
+        return ctx.ops.norm_add(residual32, y32, self.weight, self.eps, center=True, norm_scale=scale, clear=clear,
+                                rows_dtype=rows_dtype)
+
     def defer(self, ctx, x32, rows=None):
         if not hasattr(ctx.ops, "defer_layernorm"):
             return super().defer(ctx, x32, rows)

@@ -34,6 +34,7 @@ from .spec import TensorSpec
 class _MatrixMemoryMixer(Mixer):
     graph_safe = True      # launches kernels only; the state slot and the token counts are read on the device
     accepts_deferred_norm = True
+    returns_output = True
     mode = ""
 
     def __init__(self, prefix: str, width: int, n_head: int, head_dim: int, v_head_dim: int, eps: float,
@@ -74,7 +75,7 @@ class _MatrixMemoryMixer(Mixer):
         heads = ctx.ops.head_norm_gate(memory_out, aux, gate, self.norm_gain, self.n_head, self.v_head_dim,
                                        self.eps, per_head_gain, gate_activation, ctx.act_dtype,
                                        positions=ctx.positions)
-        ctx.ops.linear_residual(heads, self.out_weight, None, residual32)
+        return self.add_output(ctx, heads, self.out_weight, residual32)
 
 
 @register_mixer("gated_linear_attention")
@@ -109,7 +110,7 @@ class GatedLinearAttention(_MatrixMemoryMixer):
     def cache_spec(self):
         return FixedStateSpec((self.n_head * self.v_head_dim * self.head_dim,), "float32")
 
-    def forward(self, ctx, cache, y, residual32) -> None:
+    def forward(self, ctx, cache, y, residual32):
         ops = ctx.ops
         if hasattr(y, "materialize"):
             y = y.materialize()                      # three projections read the normalised rows
@@ -118,7 +119,7 @@ class GatedLinearAttention(_MatrixMemoryMixer):
         z = ops.linear(thin, self.decay_out, self.decay_bias, "none", torch.float32)
         out, aux = ops.matrix_memory_scan(ctx, "gla", proj, 0, self.k_off, self.v_off, self.n_head, self.head_dim,
                                           self.v_head_dim, z, self.tau, cache.state)
-        self._finish(ctx, proj, out, aux, residual32, False, "silu")
+        return self._finish(ctx, proj, out, aux, residual32, False, "silu")
 
 
 @register_mixer("mlstm")
@@ -151,7 +152,7 @@ class MLSTM(_MatrixMemoryMixer):
         # per head: head_dim x (v_head_dim + 1) numbers (the last column is the normaliser n) and the maximum m
         return FixedStateSpec((self.n_head * (self.v_head_dim + 1) * self.head_dim + self.n_head,), "float32")
 
-    def forward(self, ctx, cache, y, residual32) -> None:
+    def forward(self, ctx, cache, y, residual32):
         ops = ctx.ops
         if hasattr(y, "materialize"):
             y = y.materialize()
@@ -159,7 +160,7 @@ class MLSTM(_MatrixMemoryMixer):
         gates = ops.linear(y, self.gate_weight, self.gate_bias, "none", torch.float32)
         out, aux = ops.matrix_memory_scan(ctx, "mlstm", proj, 0, self.k_off, self.v_off, self.n_head, self.head_dim,
                                           self.v_head_dim, gates, self.gate_cap, cache.state)
-        self._finish(ctx, proj, out, aux, residual32, True, "sigmoid")
+        return self._finish(ctx, proj, out, aux, residual32, True, "sigmoid")
 
 
 @register_mixer("retention")
@@ -190,12 +191,12 @@ class Retention(_MatrixMemoryMixer):
     def cache_spec(self):
         return FixedStateSpec((self.n_head * self.v_head_dim * self.head_dim,), "float32")
 
-    def forward(self, ctx, cache, y, residual32) -> None:
+    def forward(self, ctx, cache, y, residual32):
         ops = ctx.ops
         proj = ops.linear(y, self.fused_weight, None, "none", ctx.act_dtype)
         out, aux = ops.matrix_memory_scan(ctx, "retention", proj, 0, self.k_off, self.v_off, self.n_head, self.head_dim,
                                           self.v_head_dim, None, 0.0, cache.state, head_consts=self.decays)
-        self._finish(ctx, proj, out, aux, residual32, False, "silu")
+        return self._finish(ctx, proj, out, aux, residual32, False, "silu")
 
 
 @register_mixer("wkv")

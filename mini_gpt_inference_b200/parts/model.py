@@ -33,7 +33,7 @@ class DecoderModel:
                     registry = {"norm": NORMS, "feed_forward": FEED_FORWARDS, "connection": CONNECTIONS,
                                 "side_input": SIDE_INPUTS}[role]
                     parts[name] = registry.build(part_spec, p)
-            self.layers.append(Layer(parts, roles, ARRANGEMENTS.get(layer_spec.arrangement), p))
+            self.layers.append(Layer(parts, roles, ARRANGEMENTS.get(layer_spec.arrangement), p, layer_spec.settings))
         self.entries = [STREAM_ENTRIES.build(entry, "") for entry in spec.entries]
         self.final_norm = NORMS.build(spec.final_norm, "")
         self.head = HEADS.build(spec.head, "", embedding=self.embedding)
@@ -101,6 +101,8 @@ class DecoderModel:
             layer = self.layers[call.layer]
             if call.enter is not None:
                 x = self.entries[call.enter].forward(ctx, x, x_embedded, call.enter_index)
+            if call.enter is not None or not getattr(layer.run, "keeps_stream_rows", False):
+                ctx.shared.pop("stream rows", None)      # the copy an earlier layer left is not of this stream
             x = stream_after(layer.run(ctx, layer, ctx.cache_view(call.cache_layer, call.writes_cache), x), x)
         if ctx.logit_rows.numel() == 0:
             return None

@@ -15,6 +15,12 @@ the experts of the best ``keep`` groups be chosen.  ``activation="clamped_swish"
 ``W_down (g * sigmoid(1.702 g) * (u + 1))`` with ``g = min(W_gate y, limit)``,
 ``u = clamp(W_up y, -limit, limit)``; the shared expert has a limit of its own.
 
+``gated=False`` makes an expert a plain unit, ``W_down act(W_up y)`` (``activation``: ``relu_sq``, ``gelu_tanh`` or
+``silu``; no ``gate`` tensors), and the shared expert of the same form.  Its hidden features are then cut into parts as
+large as an expert's (the last one filled up with zero rows): since ``W_down act(W_up y)`` is a sum over hidden features,
+the parts are experts that every token uses with the shared gate as their weight, and the whole feed-forward is one
+grouping and two grouped products.
+
 In the checkpoint expert ``e`` has ``e<e>.gate``, ``e<e>.up``, ``e<e>.down`` under the part's
 prefix, the router ``router``, the shared expert ``shared.gate``, ``shared.up``, ``shared.down``
 and ``shared.sg``.  When bound, the experts' matrices are stacked (``[E, 2F, C]`` with gate rows
@@ -34,19 +40,22 @@ from .spec import TensorSpec
 class RoutedExperts(FeedForward):
     graph_safe = True      # the tokens are grouped by expert on the device; the host decides nothing per step
     accepts_deferred_norm = False      # the router reads the normalised rows themselves
+    GATED, PLAIN = ("silu", "clamped_swish"), ("relu_sq", "gelu_tanh", "silu")
 
     def __init__(self, prefix: str, width: int, n_experts: int, top: int, inner: int,
                  shared_inner: int | None = None, shared_gate: bool = True, scoring: str = "softmax_top",
                  route_scale: float = 1.0, correction: bool = False, groups: tuple | None = None,
                  activation: str = "silu", limit: float = 0.0, shared_limit: float | None = None,
-                 init: str = "normal") -> None:
+                 init: str = "normal", gated: bool = True) -> None:
         super().__init__(prefix)
         if not 0 < top <= n_experts:
             raise ValueError(f"top {top} must lie in 1..n_experts ({n_experts})")
         if scoring not in ("softmax_top", "sigmoid"):
             raise ValueError(f"scoring {scoring!r}: softmax_top or sigmoid")
-        if activation not in ("silu", "clamped_swish"):
-            raise ValueError(f"activation {activation!r}: silu or clamped_swish")
+        if activation not in (self.GATED if gated else self.PLAIN):
+            raise ValueError(f"activation {activation!r}: one of {', '.join(self.GATED if gated else self.PLAIN)}")
+        if not gated and (scoring != "softmax_top" or correction or groups is not None or route_scale != 1.0):
+            raise ValueError("experts without a gate are chosen by the plain router")
         if groups is not None:
             count, keep = groups
             if n_experts % count or not 0 < keep <= count or keep * (n_experts // count) < top:
@@ -59,6 +68,10 @@ class RoutedExperts(FeedForward):
         self.correction = None
         self.width, self.n_experts, self.top, self.inner = width, n_experts, top, inner
         self.shared_inner = shared_inner
+        self.gated = bool(gated)
+        # a plain shared expert as experts that every token uses (see the module's description)
+        self.always = 0 if gated or shared_inner is None else -(-shared_inner // inner)
+        self.returns_output = not gated
         self.shared_gate = bool(shared_gate) and shared_inner is not None
         self.router = self.w_in = self.w_out = None
         self.shared_in = self.shared_out = self.shared_gate_weight = None
@@ -70,12 +83,14 @@ class RoutedExperts(FeedForward):
         if self.has_correction:
             specs[p + "correction"] = TensorSpec((self.n_experts,), "vector", "norm_shift")
         for e in range(self.n_experts):
-            specs[f"{p}e{e}.gate"] = TensorSpec((f, c), "matrix", init)
+            if self.gated:
+                specs[f"{p}e{e}.gate"] = TensorSpec((f, c), "matrix", init)
             specs[f"{p}e{e}.up"] = TensorSpec((f, c), "matrix", init)
             specs[f"{p}e{e}.down"] = TensorSpec((c, f), "matrix", init_out)
         if self.shared_inner is not None:
             s = self.shared_inner
-            specs[p + "shared.gate"] = TensorSpec((s, c), "matrix", init)
+            if self.gated:
+                specs[p + "shared.gate"] = TensorSpec((s, c), "matrix", init)
             specs[p + "shared.up"] = TensorSpec((s, c), "matrix", init)
             specs[p + "shared.down"] = TensorSpec((c, s), "matrix", init_out)
             if self.shared_gate:
@@ -88,17 +103,34 @@ class RoutedExperts(FeedForward):
             return
         self.router = tensors[p + "router"]
         self.correction = tensors.get(p + "correction") if self.has_correction else None
+        if self.shared_gate:
+            self.shared_gate_weight = tensors[p + "shared.sg"].reshape(-1).contiguous()
+        if not self.gated:
+            ups = [tensors[f"{p}e{e}.up"] for e in range(self.n_experts)]
+            downs = [tensors[f"{p}e{e}.down"] for e in range(self.n_experts)]
+            for first in range(0, self.always * self.inner, self.inner):
+                up = tensors[p + "shared.up"][first: first + self.inner]
+                down = tensors[p + "shared.down"][:, first: first + self.inner]
+                fill = self.inner - up.shape[0]
+                ups.append(torch.nn.functional.pad(up, (0, 0, 0, fill)))
+                downs.append(torch.nn.functional.pad(down, (0, fill)))
+            self.w_in, self.w_out = torch.stack(ups).contiguous(), torch.stack(downs).contiguous()
+            return
         self.w_in = torch.stack([torch.cat([tensors[f"{p}e{e}.gate"], tensors[f"{p}e{e}.up"]], dim=0)
                                  for e in range(self.n_experts)]).contiguous()
         self.w_out = torch.stack([tensors[f"{p}e{e}.down"] for e in range(self.n_experts)]).contiguous()
         if self.shared_inner is not None:
             self.shared_in = torch.cat([tensors[p + "shared.gate"], tensors[p + "shared.up"]], dim=0).contiguous()
             self.shared_out = tensors[p + "shared.down"]
-            if self.shared_gate:
-                self.shared_gate_weight = tensors[p + "shared.sg"].reshape(-1).contiguous()
 
-    def forward(self, ctx, y, residual32) -> None:
+    def forward(self, ctx, y, residual32):
         ops = ctx.ops
+        if not self.gated:
+            ids, weights, _ = ops.moe_route(y, self.router, self.shared_gate_weight, ctx.positions, self.top, always=self.always)
+            if residual32 is None:
+                return ops.moe_experts(y, ids, weights, self.w_in, self.w_out, activation=self.activation, gated=False)
+            ops.moe_experts_residual(y, ids, weights, self.w_in, self.w_out, residual32, activation=self.activation, gated=False)
+            return None
         if self.scoring == "softmax_top" and not self.has_correction and self.groups is None:
             ids, weights, gate = ops.moe_route(y, self.router, self.shared_gate_weight, ctx.positions, self.top)
             if self.route_scale != 1.0:

@@ -32,10 +32,12 @@ class RMSNorm(Norm):
     def forward(self, ctx, x32):
         return ctx.ops.rmsnorm(x32, self.weight, self.eps, self.offset, ctx.act_dtype)
 
-    def add_normed(self, ctx, y32, residual32, clear=False):
-        """``residual32 += norm(y32)`` in 32-bit, in place: the norm behind a sublayer.  ``clear``: ``y32`` is left
-        as zeros (a buffer that the next sublayer adds into)."""
-        return ctx.ops.rmsnorm_add(residual32, y32, self.weight, self.eps, self.offset, clear=clear)
+    def add_normed(self, ctx, y32, residual32, clear=False, scale=1.0, rows_dtype=None):
+        """``residual32 += scale * norm(y32)`` in 32-bit, in place: the norm behind a sublayer.  ``clear``: ``y32`` is left
+        as zeros (a buffer that the next sublayer adds into).  With ``rows_dtype`` the new stream is also returned in
+        that type."""
+        return ctx.ops.norm_add(residual32, y32, self.weight, self.eps, self.offset, norm_scale=scale, clear=clear,
+                                rows_dtype=rows_dtype)
 
     def defer(self, ctx, x32, rows=None):
         if not hasattr(ctx.ops, "defer_rmsnorm"):

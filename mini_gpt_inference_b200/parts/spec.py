@@ -34,6 +34,7 @@ class LayerSpec:
     prefix: str                             # weight-name prefix of the layer ("blocks.0.")
     parts: Mapping[str, PartSpec]           # name in the layer -> part
     arrangement: str = "pre_norm"           # key in the block-arrangement registry
+    settings: Mapping[str, Any] = field(default_factory=dict)   # numbers of the arrangement itself
 
     def role_of(self, name: str) -> str:
         role = self.parts[name].role

@@ -145,13 +145,18 @@ class TorchOps:
             out = out * torch.sigmoid(gate.float())
         return out.to(q.dtype)
 
-    def moe_route(self, y, router_weight, gate_weight, positions, top):
+    def moe_route(self, y, router_weight, gate_weight, positions, top, always=0):
         z = y.float() @ router_weight.float().T
         vals, ids = torch.topk(z, top, dim=-1)
         weights = torch.softmax(vals, dim=-1)
+        gate = torch.sigmoid(y.float() @ gate_weight.float()) if gate_weight is not None else None
+        if always:
+            extra = torch.arange(z.shape[1], z.shape[1] + always).expand(len(z), always)
+            ids = torch.cat([ids, extra], dim=-1)
+            share = torch.ones(len(z)) if gate is None else gate
+            weights, gate = torch.cat([weights, share[:, None].expand(len(z), always)], dim=-1), None
         ids = ids.to(torch.int32)
         ids[positions < 0] = -1
-        gate = torch.sigmoid(y.float() @ gate_weight.float()) if gate_weight is not None else None
         return ids, weights, gate
 
     @staticmethod
@@ -165,16 +170,31 @@ class TorchOps:
             return a * torch.sigmoid(1.702 * a) * (u + 1.0)
         raise ValueError(activation)
 
-    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0):
-        inner = w_in.shape[1] // 2
+    @staticmethod
+    def _plain(z, activation):
+        if activation == "relu_sq":
+            return z.clamp(min=0.0) ** 2
+        if activation == "gelu_tanh":
+            return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+        if activation == "silu":
+            return z * torch.sigmoid(z)
+        raise ValueError(activation)
+
+    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0, gated=True):
+        inner = w_out.shape[2]
         for t in range(y.shape[0]):
             for k in range(ids.shape[1]):
                 e = int(ids[t, k])
                 if e < 0:
                     continue
                 a = w_in[e].float() @ y[t].float()
-                hidden = self._gated(a[:inner], a[inner:], activation, limit).to(y.dtype).float()
-                residual32[t] += weights[t, k] * (w_out[e].float() @ hidden)
+                hidden = self._gated(a[:inner], a[inner:], activation, limit) if gated else self._plain(a, activation)
+                residual32[t] += weights[t, k] * (w_out[e].float() @ hidden.to(y.dtype).float())
+
+    def moe_experts(self, y, ids, weights, w_in, w_out, activation="silu", limit=0.0, gated=True):
+        out = torch.zeros(y.shape[0], w_out.shape[1])
+        self.moe_experts_residual(y, ids, weights, w_in, w_out, out, activation, limit, gated)
+        return out
 
     def moe_route_scored(self, y, router_weight, gate_weight, positions, top, scoring, correction, groups, scale):
         z = y.float() @ router_weight.float().T
@@ -416,15 +436,28 @@ class TorchOps:
             cache.k_pages[page, :, off] = k[keep].to(cache.k_pages.dtype)
             cache.v_pages[page, :, off] = v[keep].to(cache.v_pages.dtype)
 
-    def latent_prepare(self, proj, n_head, q_off, q_dim, rot_dim, low_off, rank, gain, eps, freq, cache, slots, positions):
+    def _turn_any(self, x, positions, rot_dims, freq, neighbours, magnitude):
+        """All ``rot_dims`` features turn; pairs are halves or neighbours."""
+        if rot_dims == 0:
+            return x
+        if not neighbours:
+            return magnitude * self._turn(x, positions, rot_dims, freq)
+        order = torch.cat([torch.arange(0, rot_dims, 2), torch.arange(1, rot_dims, 2)])
+        out = torch.empty_like(x)
+        out[..., order] = magnitude * self._turn(x[..., order], positions, rot_dims, freq)
+        return out
+
+    def latent_prepare(self, proj, n_head, q_off, q_dim, rot_dim, low_off, rank, gain, eps, freq, cache, slots, positions,
+                       neighbours=False, magnitude=1.0):
         n = proj.shape[0]
         q_in = proj[:, q_off: q_off + n_head * (q_dim + rot_dim)].float().reshape(n, n_head, q_dim + rot_dim)
         q = torch.zeros(n, n_head, rank + rot_dim)
-        q[..., rank:] = self._turn(q_in[..., q_dim:], positions, rot_dim, freq)
+        q[..., rank:] = self._turn_any(q_in[..., q_dim:], positions, rot_dim, freq, neighbours, magnitude)
         if cache is not None and cache.writes:
             c = proj[:, low_off: low_off + rank].float()
             c = c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * gain
-            shared = self._turn(proj[:, None, low_off + rank: low_off + rank + rot_dim].float(), positions, rot_dim, freq)[:, 0]
+            shared = self._turn_any(proj[:, None, low_off + rank: low_off + rank + rot_dim].float(), positions, rot_dim, freq,
+                                    neighbours, magnitude)[:, 0]
             keep = (positions >= 0) & (slots >= 0)
             page, off = slots[keep].long() // cache.page_tokens, slots[keep].long() % cache.page_tokens
             cache.k_pages[page, 0, off] = torch.cat([c, shared], dim=-1)[keep].to(cache.k_pages.dtype)
@@ -539,13 +572,20 @@ class TorchOps:
             shared[key] = out
         return out
 
-    def rmsnorm_add(self, residual32, y32, weight, eps, offset=0.0, other32=None, scale=1.0, other_scale=1.0, clear=False):
+    def norm_add(self, residual32, y32, weight, eps, offset=0.0, center=False, norm_scale=1.0, other32=None, scale=1.0,
+                 other_scale=1.0, clear=False, rows_dtype=None):
         y = scale * y32 if other32 is None else scale * y32 + other_scale * other32
-        residual32 += y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * (offset + weight)
+        if center:
+            y = y - y.mean(-1, keepdim=True)
+        residual32 += norm_scale * (y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * (offset + weight))
         if clear:
             y32.zero_()
             if other32 is not None:
                 other32.zero_()
+        return None if rows_dtype is None else residual32.to(rows_dtype)
+
+    def rmsnorm_add(self, residual32, y32, weight, eps, offset=0.0, other32=None, scale=1.0, other_scale=1.0, clear=False):
+        self.norm_add(residual32, y32, weight, eps, offset, other32=other32, scale=scale, other_scale=other_scale, clear=clear)
         return residual32
 
     def add_rows(self, x32, rows32, vector):
