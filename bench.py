@@ -30,6 +30,8 @@ mixed with a loop and routed experts) beside the two other designs at equal size
 four; then the kinds mixed) beside Zenedra's closest layers at equal sizes.
 ``--only lunelorn`` likewise: the Lunelorn decoder (layers of one mixer kind each with routed experts, then the
 kinds mixed with a loop and the per-layer token input) beside Zenedra's closest layers at equal sizes.
+``--only nogatar`` likewise: the Nogatar decoder (layers of one mixer kind each with routed experts, then both kinds
+mixed) beside Nukodra's latent attention, Zenedra's mLSTM and Lunelorn's routed experts at equal sizes.
 ``--only designs`` prints a line of its own: the Fakilorn decoder beside this decoder at equal width,
 depth, hidden width and vocabulary (random weights, two sizes): a 2,048-token prompt step, decode
 steps at the headline batch with contexts near 2,048, and the device time of every exported function
@@ -93,7 +95,7 @@ def parse_args():
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--page-tokens", type=int, default=64)
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and prefill")
-    ap.add_argument("--only", choices=["all", "decode", "prefill", "serve", "kernels", "designs", "zenedra", "nukodra", "lunelorn"], default="all",
+    ap.add_argument("--only", choices=["all", "decode", "prefill", "serve", "kernels", "designs", "zenedra", "nukodra", "lunelorn", "nogatar"], default="all",
                     help="a small case for profilers: only the device-timed decode steps, or only "
                          "the 2,048-token prefill (the printed line is then partial); serve: 64 "
                          "requests with prompts of 16 to 512 tokens and 256 generated tokens each "
@@ -741,6 +743,53 @@ def compare_lunelorn(args) -> dict:
     return out
 
 
+# ``--only nogatar``: the Nogatar decoder beside the closest layers here at equal width, depth, head count and vocabulary
+# (random weights): Nukodra's attention over cached latents (the same projections, preparation and attention kernels;
+# gated dense feed-forwards), Zenedra's mLSTM (the same scan and chunk kernels) and Lunelorn's routed experts in every
+# layer.  Layers of one mixer kind each: latents of 512 with heads of 128 + 64 features, neighbouring features rotated
+# with stretched frequencies, a sink, without a window and with one of 512; mLSTM with half as many heads and values of
+# 128.  Feed-forwards are routed experts without a gate and a shared one (as wide as an expert; in the larger size, two
+# experts wide) throughout (the design has no dense one).  Then the kinds mixed, three attention layers to one mLSTM.
+def _nogatar_raw(sz: dict, kinds: list, window) -> dict:
+    heads = sz["heads"]
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+              "rot": {"dims": 64, "base": 10000.0, "scaling": {"factor": 4.0, "original": 512, "fast": 32.0, "slow": 1.0}}}
+    if window:
+        latent["mask"] = {"size": window}
+    mixers = {"latent_attention": latent, "mlstm": {"heads": heads // 2, "dim": 64, "vdim": 128, "gate_cap": 10.0}}
+    routed = {"kind": "moe", "expert": {"ff": sz["expert_ff"]}, "router": {"experts": sz["experts"], "top": sz["top"]},
+              "shared": {"ff": sz["shared_ff"]}}
+    return {"architecture": "Nogatar", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": sz["width"] ** 0.5}, "residual_mult": 0.5, "logit_softcap": 30.0,
+            "layers": [{"type": kind, "mixer": dict(mixers[kind]), "mlp": routed} for kind in kinds]}
+
+
+def compare_nogatar(args) -> dict:
+    import torch
+
+    from mini_gpt_inference_b200 import LunelornConfig, NogatarConfig, NukodraConfig, ZenedraConfig
+    from mini_gpt_inference_b200.kernels.ops import default_ops
+
+    ops = default_ops("cuda:0")
+    batch, context, prompt_len = args.batch, 2048, PREFILL_TOKENS
+    flush = torch.empty(256 * 1024 * 1024, dtype=torch.uint8, device="cuda:0")
+    out = {"impl": "ours", "partial": "nogatar beside nukodra, zenedra and lunelorn", "dtype": args.dtype, "batch": batch,
+           "context": context, "prompt": prompt_len, "rows": []}
+    for size_name, sz in DESIGN_SIZES.items():
+        n = sz["layers"]
+        mixed = (["latent_attention", "mlstm", "latent_attention", "latent_attention"] * n)[:n]
+        for name, cfg in (
+                ("nukodra {} latent attention, dense", NukodraConfig.from_dict(_nukodra_raw(sz, ["latent_attention"] * n, None))),
+                ("zenedra {} mlstm, dense", ZenedraConfig.from_dict(_zenedra_raw(sz, ["mlstm"] * n, False, False, context))),
+                ("lunelorn {} retention, experts", LunelornConfig.from_dict(_lunelorn_raw(sz, ["retention"] * n, None, False))),
+                ("nogatar {} latent attention, experts", NogatarConfig.from_dict(_nogatar_raw(sz, ["latent_attention"] * n, None))),
+                ("nogatar {} latent attention, window 512, experts", NogatarConfig.from_dict(_nogatar_raw(sz, ["latent_attention"] * n, 512))),
+                ("nogatar {} mlstm, experts", NogatarConfig.from_dict(_nogatar_raw(sz, ["mlstm"] * n, None))),
+                ("nogatar {} mixed, window 512, experts", NogatarConfig.from_dict(_nogatar_raw(sz, mixed, 512)))):
+            out["rows"].append(_measure_design(args, ops, flush, name.format(size_name), cfg, batch, context, prompt_len))
+    return out
+
+
 def check_decode_logits(args) -> dict:
     """Outside every timed region: the decode step that the benchmark times (batch 8, contexts of
     2,048, the replayed graph) is run once on fixed tokens and its logits are compared with rows
@@ -808,6 +857,8 @@ def run_ours(args) -> dict:
         return compare_nukodra(args)
     if args.only == "lunelorn":
         return compare_lunelorn(args)
+    if args.only == "nogatar":
+        return compare_nogatar(args)
     if args.only == "decode":
         cfg, windows, launches, mean_ctx, clocks = device_decode(args, args.batch, args.steps, args.warmup,
                                                                  min_seconds=0.0)

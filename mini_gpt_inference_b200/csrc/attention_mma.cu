@@ -677,14 +677,12 @@ attention_wide_kernel(const AttnParams p, const int single, const int dpad, cons
     };
     load_keys(j_first, kbuf);
     cp_async_commit();
+    if (j_first + KB <= j_last) load_keys(j_first + KB, kbuf + KB * stride);
+    cp_async_commit();
     int buf = 0;
     for (int j0 = j_first; j0 <= j_last; j0 += KB, buf ^= 1) {
-        cp_async_wait<0>();
-        __syncthreads();                                   // the block is here; everyone has left the one before
-        if (j0 + KB <= j_last) {
-            load_keys(j0 + KB, kbuf + (buf ^ 1) * KB * stride);
-            cp_async_commit();
-        }
+        cp_async_wait<1>();                                // (one group a block, empty ones behind the last)
+        __syncthreads();                                   // the block is here, for everyone
         const bf16* kb = kbuf + buf * KB * stride;
         float s[2][4];
 #pragma unroll
@@ -769,6 +767,9 @@ attention_wide_kernel(const AttnParams p, const int single, const int dpad, cons
                 mma16816(o[n + 1], a, b[2], b[3]);
             }
         }
+        __syncthreads();                                   // everyone has left the buffer: it takes the block after the next
+        if (j0 + 2 * KB <= j_last) load_keys(j0 + 2 * KB, kbuf + buf * KB * stride);
+        cp_async_commit();
     }
     // the four warps of a row group kept the sums of their own keys: they meet here
     __syncthreads();
@@ -823,7 +824,7 @@ int launch_wide(const AttnParams& p, int single, int n_tiles, int dpad, size_t s
         e = mg_launch(attention_wide_kernel<CW>, grid, dim3(256), smem, s, true, p, single, dpad, row_tiles);
     }
     if (e == cudaSuccess && single)
-        e = mg_launch(attention_merge_kernel, dim3(p.n_tokens, p.n_head), dim3(128), 0, s, true, p);
+        e = mg_launch(attention_merge_kernel, dim3(p.n_tokens, p.n_head), dim3(p.dv > 256 ? 512 : p.dv > 128 ? 256 : 128), 0, s, true, p);
     if (e != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "attention (wide rows): %s", cudaGetErrorString(e));
     return MG_OK;
 }

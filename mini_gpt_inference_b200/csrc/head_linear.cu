@@ -169,6 +169,92 @@ head_linear_mma_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_he
     }
 }
 
+// bfloat16 with up to 16 tokens: a CTA owns 16 outputs of one head.  Its part of the head's matrix does not depend on
+// the kernel before, so all of it is asked for (cp.async) before the dependency wait, and the tokens' inputs right
+// behind it: one trip to memory, whatever I is.  The four warps take the 16-wide steps of i in turn; their sums meet in
+// shared memory and are added in the warps' order.
+constexpr int FEW = 16, FEW_OUT = 16;
+constexpr size_t few_smem(int I, int rows_are_inputs) {
+    const size_t ip = (size_t)(I + 15) / 16 * 16;
+    return sizeof(bf16) * (FEW * (ip + MPAD) + (rows_are_inputs ? ip * (FEW_OUT + MPAD) : FEW_OUT * (ip + MPAD)));
+}
+
+__device__ __forceinline__ void hl_copy16(bf16* dst, const bf16* src, bool real) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    const int bytes = real ? 16 : 0;                       // 0: nothing is read, the 16 bytes become zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(bytes) : "memory");
+}
+
+__global__ void __launch_bounds__(128)
+head_linear_few_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_head, const bf16* __restrict__ w,
+                       int rows_are_inputs, const bf16* __restrict__ gate, int gate_ld, bf16* __restrict__ out, int out_ld,
+                       int out_off, int out_head, int n_tokens, int I, int J) {
+    extern __shared__ __align__(16) uint8_t few_raw[];
+    __shared__ float part[4][FEW][FEW_OUT];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, j0 = blockIdx.y * FEW_OUT;
+    const int ip = (I + 15) / 16 * 16, xs_ld = ip + MPAD, ws_ld = rows_are_inputs ? FEW_OUT + MPAD : ip + MPAD;
+    bf16* xs = reinterpret_cast<bf16*>(few_raw);           // [16][ip + 8]
+    bf16* ws = xs + FEW * xs_ld;                           // [16 outputs][ip + 8], or [ip][16 outputs + 8]
+    const bf16* wh = w + (size_t)h * I * J;
+    if (rows_are_inputs) {
+        for (int idx = tid; idx < ip * 2; idx += 128) {
+            const int i = idx >> 1, c = (idx & 1) * 8;
+            const bool real = i < I && j0 + c < J;
+            hl_copy16(ws + i * ws_ld + c, real ? wh + (size_t)i * J + j0 + c : w, real);
+        }
+    } else {
+        const int chunks = ip >> 3;
+        for (int idx = tid; idx < FEW_OUT * chunks; idx += 128) {
+            const int r = idx / chunks, c = (idx - r * chunks) * 8;
+            const bool real = j0 + r < J && c < I;
+            hl_copy16(ws + r * ws_ld + c, real ? wh + (size_t)(j0 + r) * I + c : w, real);
+        }
+    }
+    pdl_trigger();
+    pdl_wait();
+    {
+        const int chunks = ip >> 3;
+        const bf16* xh = x + x_off + (size_t)h * x_head;
+        for (int idx = tid; idx < FEW * chunks; idx += 128) {
+            const int t = idx / chunks, c = (idx - t * chunks) * 8;
+            const bool real = t < n_tokens && c < I;
+            hl_copy16(xs + t * xs_ld + c, real ? xh + (size_t)t * x_ld + c : x, real);
+        }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    float acc[2][4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[0][e] = acc[1][e] = 0.f;
+    for (int kk = warp * 16; kk < ip; kk += 64) {
+        uint32_t a[4], b[4];
+        hl_ldsm(a, xs + (lane & 15) * xs_ld + kk + (lane >> 4) * 8);
+        if (rows_are_inputs) hl_ldsm_t(b, ws + (kk + ((lane >> 3) & 1) * 8 + (lane & 7)) * ws_ld + (lane >> 4) * 8);
+        else hl_ldsm(b, ws + ((lane >> 4) * 8 + (lane & 7)) * ws_ld + kk + ((lane >> 3) & 1) * 8);
+        hl_mma(acc[0], a, b[0], b[1]);
+        hl_mma(acc[1], a, b[2], b[3]);
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) part[warp][(lane >> 2) + 8 * (e >> 1)][t * 8 + 2 * (lane & 3) + (e & 1)] = acc[t][e];
+    __syncthreads();
+    for (int idx = tid; idx < FEW * FEW_OUT / 2; idx += 128) {
+        const int n = idx >> 3, c = (idx & 7) * 2, j = j0 + c;
+        if (n >= n_tokens || j >= J) continue;
+        float v[2];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) v[u] = (part[0][n][c + u] + part[1][n][c + u]) + (part[2][n][c + u] + part[3][n][c + u]);
+        if (gate) {
+            const __nv_bfloat162 g = *reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)n * gate_ld + (size_t)h * J + j);
+            v[0] *= 1.0f / (1.0f + expf(-__bfloat162float(g.x)));
+            v[1] *= 1.0f / (1.0f + expf(-__bfloat162float(g.y)));
+        }
+        *reinterpret_cast<__nv_bfloat162*>(out + (size_t)n * out_ld + out_off + (size_t)h * out_head + j) = __floats2bfloat162_rn(v[0], v[1]);
+    }
+}
+
 }  // namespace
 
 // x: rows of x_ld elements, head h's I inputs from column x_off + h * x_head; w: [n_head * J, I] or, if
@@ -189,6 +275,21 @@ MG_API int mg_head_linear(const void* x, int x_ld, int x_off, int x_head, const 
     const bool vectors = I % 8 == 0 && J % 8 == 0 && x_ld % 8 == 0 && x_off % 8 == 0 && x_head % 8 == 0 && out_ld % 2 == 0 &&
                          out_off % 2 == 0 && out_head % 2 == 0 && gate_ld % 2 == 0 && (uintptr_t)x % 16 == 0 &&
                          (uintptr_t)w % 16 == 0 && (uintptr_t)out % 4 == 0 && (uintptr_t)gate % 4 == 0;
+    if (is_bf16 && vectors && n_tokens <= FEW && few_smem(I, rows_are_inputs) <= 96 * 1024) {
+        static bool configured = false;
+        if (!configured) {
+            const cudaError_t ec = cudaFuncSetAttribute(head_linear_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+            if (ec != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "head_linear (shared memory): %s", cudaGetErrorString(ec));
+            configured = true;
+        }
+        MG_REQUIRE(ceil_div(J, FEW_OUT) <= 65535, "head_linear: too many outputs");
+        const cudaError_t ef = mg_launch(head_linear_few_kernel, dim3(n_head, ceil_div(J, FEW_OUT)), dim3(128),
+                                         few_smem(I, rows_are_inputs), s, true, (const bf16*)x, x_ld, x_off, x_head, (const bf16*)w,
+                                         rows_are_inputs, (const bf16*)gate, gate_ld, (bf16*)out, out_ld, out_off, out_head,
+                                         n_tokens, I, J);
+        if (ef != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "head_linear (few tokens): %s", cudaGetErrorString(ef));
+        return MG_OK;
+    }
     if (is_bf16 && vectors) {
         const int mn = n_tokens <= 32 ? 16 : 64;
         const dim3 tiles(ceil_div(n_tokens, MT), n_head, ceil_div(J, mn));

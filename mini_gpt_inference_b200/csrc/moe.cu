@@ -22,61 +22,87 @@ MG_GUARD_DECLARE(moe)
 namespace {
 
 // ---- router ------------------------------------------------------------------------------------
-// One CTA per token: its warps share the experts (and the gate, as one more row of weights), a lane
-// sums every 32nd group of four features in a fixed order, so a token's logits depend on nothing
-// but the token.  Warp 0 then picks the `top` largest one after the other.
-constexpr int ROUTE_WARPS = 8;
+// A CTA takes one token, or, in steps of many, ROUTE_TOKENS neighbours that share every read of the router's rows: its
+// warps share the experts (and the gate, as one more row of weights), a lane sums every 32nd group of four features in a
+// fixed order, so a token's logits depend on nothing but the token.  A warp per token then picks the `top` largest one
+// after the other.
+constexpr int ROUTE_WARPS = 8, ROUTE_TOKENS = 4;
+constexpr int ROUTE_WARPS_FEW = 24;      // steps of few tokens: a warp per expert as far as they reach, so that all rows' reads are in flight at once
+
+__device__ __forceinline__ float4 route_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 route_load4(const bf16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// dot[u] = row_u . wr for NT rows of `width` features that lie one after the other
+template <typename T, int NT>
+__device__ __forceinline__ void route_dots(float (&dot)[NT], const T* __restrict__ rows, const float* __restrict__ wr, int width,
+                                           int lane, bool vec) {
+#pragma unroll
+    for (int u = 0; u < NT; ++u) dot[u] = 0.f;
+    if (vec) {
+#pragma unroll (NT == 1 ? 8 : 4)
+        for (int c = lane * 4; c < width; c += 128) {
+            const float4 wv = route_load4(wr + c);
+#pragma unroll
+            for (int u = 0; u < NT; ++u) {
+                const float4 r = route_load4(rows + (size_t)u * width + c);
+                dot[u] = fmaf(r.x, wv.x, dot[u]);
+                dot[u] = fmaf(r.y, wv.y, dot[u]);
+                dot[u] = fmaf(r.z, wv.z, dot[u]);
+                dot[u] = fmaf(r.w, wv.w, dot[u]);
+            }
+        }
+    } else {
+        for (int c = lane; c < width; c += 32)
+#pragma unroll
+            for (int u = 0; u < NT; ++u) dot[u] = fmaf(to_float(rows[(size_t)u * width + c]), wr[c], dot[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < NT; ++u) dot[u] = warp_sum(dot[u]);
+}
 
 template <typename T>
 __device__ __forceinline__ float route_dot(const T* __restrict__ row, const float* __restrict__ wr, int width, int lane,
                                            bool vec) {
-    float dot = 0.f;
-    if (vec) {
-#pragma unroll 4
-        for (int c = lane * 4; c < width; c += 128) {
-            const float4 wv = *reinterpret_cast<const float4*>(wr + c);
-            dot = fmaf(to_float(row[c]), wv.x, dot);
-            dot = fmaf(to_float(row[c + 1]), wv.y, dot);
-            dot = fmaf(to_float(row[c + 2]), wv.z, dot);
-            dot = fmaf(to_float(row[c + 3]), wv.w, dot);
-        }
-    } else {
-        for (int c = lane; c < width; c += 32) dot = fmaf(to_float(row[c]), wr[c], dot);
-    }
-    return warp_sum(dot);
+    float dot[1];
+    route_dots<T, 1>(dot, row, wr, width, lane, vec);
+    return dot[0];
 }
 
-template <typename T>
-__global__ void __launch_bounds__(32 * ROUTE_WARPS)
+template <typename T, int NT, int WARPS>
+__global__ void __launch_bounds__(32 * WARPS)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ w_gate,
                  const int* __restrict__ positions, int* __restrict__ ids, float* __restrict__ weights,
                  float* __restrict__ gate, int n_tokens, int width, int n_experts, int top, int always) {
-    extern __shared__ float z[];                           // [n_experts], then the gate
+    extern __shared__ float z_all[];                       // per token: [n_experts], then the gate
     pdl_trigger();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int token = blockIdx.x;
-    if (positions != nullptr && positions[token] < 0) {    // padding of a fixed-size batch: no expert
-        for (int k = threadIdx.x; k < top + always; k += blockDim.x) {
-            ids[(size_t)token * (top + always) + k] = -1;
-            weights[(size_t)token * (top + always) + k] = 0.f;
-        }
-        if (gate != nullptr && threadIdx.x == 0) gate[token] = 0.f;
-        return;
-    }
-    const T* row = h + (size_t)token * width;
-    const bool vec = width % 4 == 0 && ((uintptr_t)w_router % 16 == 0) && (w_gate == nullptr || (uintptr_t)w_gate % 16 == 0);
+    const bool vec = width % 4 == 0 && ((uintptr_t)w_router % 16 == 0) && (uintptr_t)h % 16 == 0 && (w_gate == nullptr || (uintptr_t)w_gate % 16 == 0);
     const int rows = n_experts + (w_gate != nullptr ? 1 : 0);
-    ids += (size_t)token * (top + always), weights += (size_t)token * (top + always);
-    for (int e = warp; e < rows; e += ROUTE_WARPS) {
-        const float dot = route_dot(row, e < n_experts ? w_router + (size_t)e * width : w_gate, width, lane, vec);
-        if (lane == 0) {
-            if (e < n_experts) z[e] = dot;
-            else z[e] = 1.0f / (1.0f + expf(-dot));
-        }
+    const int first = min((int)blockIdx.x * NT, n_tokens - NT);        // (the last CTA may reach back; see below)
+    for (int e = warp; e < rows; e += WARPS) {
+        float dot[NT];
+        route_dots<T, NT>(dot, h + (size_t)first * width, e < n_experts ? w_router + (size_t)e * width : w_gate, width, lane, vec);
+        if (lane == 0)
+#pragma unroll
+            for (int u = 0; u < NT; ++u)
+                z_all[u * (n_experts + 1) + e] = e < n_experts ? dot[u] : 1.0f / (1.0f + expf(-dot[u]));
     }
     __syncthreads();
-    if (warp != 0) return;
+    const int token = first + warp;
+    if (warp >= NT || token < (int)blockIdx.x * NT) return;            // tokens reached back to are the CTA's before
+    float* z = z_all + warp * (n_experts + 1);
+    ids += (size_t)token * (top + always), weights += (size_t)token * (top + always);
+    if (positions != nullptr && positions[token] < 0) {    // padding of a fixed-size batch: no expert
+        for (int k = lane; k < top + always; k += 32) ids[k] = -1, weights[k] = 0.f;
+        if (gate != nullptr && lane == 0) gate[token] = 0.f;
+        return;
+    }
     if (gate != nullptr && lane == 0) gate[token] = z[n_experts];
     // experts that every token uses, behind the chosen ones
     for (int k = lane; k < always; k += 32) {
@@ -151,7 +177,7 @@ moe_route_scored_kernel(const T* __restrict__ h, const float* __restrict__ w_rou
         return;
     }
     const T* row = h + (size_t)token * width;
-    const bool vec = width % 4 == 0 && ((uintptr_t)w_router % 16 == 0) && (w_gate == nullptr || (uintptr_t)w_gate % 16 == 0);
+    const bool vec = width % 4 == 0 && ((uintptr_t)w_router % 16 == 0) && (uintptr_t)h % 16 == 0 && (w_gate == nullptr || (uintptr_t)w_gate % 16 == 0);
     const int rows = n_experts + (gate != nullptr ? 1 : 0);
     for (int e = warp; e < rows; e += ROUTE_WARPS) {
         const float dot = route_dot(row, e < n_experts ? w_router + (size_t)e * width : w_gate, width, lane, vec);
@@ -635,16 +661,23 @@ MG_API int mg_moe_route(const void* h, const float* w_router, const float* w_gat
     MG_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top > 0 && top <= n_experts, "moe route: bad sizes");
     MG_REQUIRE(gate == nullptr || w_gate != nullptr, "moe route: a gate wants its weights");
     MG_REQUIRE(always >= 0 && (w_gate == nullptr || gate != nullptr || always > 0), "moe route: a gate that nothing takes");
-    const size_t smem = (size_t)(n_experts + 1) * sizeof(float);
+    const int per = n_tokens >= 2 * 148 * ROUTE_TOKENS ? ROUTE_TOKENS : 1;        // many tokens: still two CTAs an SM
+    const int warps = n_tokens <= 148 ? ROUTE_WARPS_FEW : ROUTE_WARPS;
+    const size_t smem = (size_t)per * (n_experts + 1) * sizeof(float);
     MG_REQUIRE(smem <= 48 * 1024, "moe route: too many experts (%d)", n_experts);
-    const dim3 grid(n_tokens), block(32 * ROUTE_WARPS);
+    const dim3 grid(ceil_div(n_tokens, per)), block(32 * warps);
     cudaError_t e;
-    if (is_bf16)
-        e = mg_launch(moe_route_kernel<bf16>, grid, block, smem, (cudaStream_t)stream, true, (const bf16*)h, w_router,
-                      w_gate, positions, ids, weights, gate, n_tokens, width, n_experts, top, always);
-    else
-        e = mg_launch(moe_route_kernel<float>, grid, block, smem, (cudaStream_t)stream, true, (const float*)h, w_router,
-                      w_gate, positions, ids, weights, gate, n_tokens, width, n_experts, top, always);
+    if (is_bf16) {
+        auto kernel = per != 1 ? moe_route_kernel<bf16, ROUTE_TOKENS, ROUTE_WARPS>
+                    : warps == ROUTE_WARPS ? moe_route_kernel<bf16, 1, ROUTE_WARPS> : moe_route_kernel<bf16, 1, ROUTE_WARPS_FEW>;
+        e = mg_launch(kernel, grid, block, smem, (cudaStream_t)stream, true, (const bf16*)h, w_router, w_gate, positions, ids,
+                      weights, gate, n_tokens, width, n_experts, top, always);
+    } else {
+        auto kernel = per != 1 ? moe_route_kernel<float, ROUTE_TOKENS, ROUTE_WARPS>
+                    : warps == ROUTE_WARPS ? moe_route_kernel<float, 1, ROUTE_WARPS> : moe_route_kernel<float, 1, ROUTE_WARPS_FEW>;
+        e = mg_launch(kernel, grid, block, smem, (cudaStream_t)stream, true, (const float*)h, w_router, w_gate, positions, ids,
+                      weights, gate, n_tokens, width, n_experts, top, always);
+    }
     MG_LAUNCHED(e, "moe route");
     return MG_OK;
 }

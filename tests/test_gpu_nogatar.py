@@ -127,7 +127,7 @@ def test_latent_rows_with_neighbouring_features_turned(ops, dtype, heads, q_dim,
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("tokens", [1, 5, 64, 65, 200])
+@pytest.mark.parametrize("tokens", [1, 5, 64, 65, 200, 1187])
 @pytest.mark.parametrize("experts,top,width,inner,shared", [(5, 2, 64, 40, 40), (4, 1, 96, 48, None), (3, 3, 72, 20, 50),
                                                             (16, 4, 128, 128, 64), (2, 1, 70, 33, 33)])
 def test_router_and_experts_without_a_gate(ops, dtype, tokens, experts, top, width, inner, shared):
