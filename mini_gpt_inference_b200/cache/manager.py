@@ -6,7 +6,8 @@ otherwise) and every request has one block table per group, shared by
 the group's layers — the same page id indexes every layer's storage, as in the
 reference (src/minigpt_infer/cache/paged.py:122-123, 154-155).  Pages are given back
 when a request is released (src/minigpt_infer/cache/paged.py:79-81) or, in a group with
-a window, as soon as no later query can read them.  A request also holds one slot of
+a window, as soon as no later query can read them (the pages of first tokens that stay in sight, ``keep_first``, are
+kept).  A request also holds one slot of
 the state pool from admission to release, whether or not any layer keeps state.
 
 Growth is asked for in two halves so that a caller can back out: ``reserve`` takes the
@@ -107,6 +108,11 @@ class CacheManager:
         bounds = [b for b in (spec.window, spec.block) if b is not None]
         return min(bounds) if bounds else None
 
+    @staticmethod
+    def _kept_pages(spec: PagedKVSpec, page_tokens: int) -> int:
+        """Pages at a sequence's start that are never given back before its end."""
+        return (spec.keep_first + page_tokens - 1) // page_tokens
+
     def _geometry(self, spec: PagedKVSpec) -> tuple[int, int]:
         pt = spec.page_tokens or self.page_tokens
         if spec.num_pages is not None:
@@ -116,7 +122,7 @@ class CacheManager:
         if self._reach(spec) is not None and self.window_slack_tokens is not None:
             # pages a request can hold at once: the window, the tokens of one step, and the two
             # pages that the window's and the portion's ends share with their neighbours
-            per_request = (self._reach(spec) + self.window_slack_tokens + pt - 1) // pt + 2
+            per_request = (self._reach(spec) + self.window_slack_tokens + pt - 1) // pt + 2 + self._kept_pages(spec, pt)
             pages = min(pages, self.max_requests * per_request)
         return pt, pages
 
@@ -136,13 +142,14 @@ class CacheManager:
             need = group.pages_for(num_tokens)
             if self._reach(group.spec) is not None:
                 slack = self.window_slack_tokens if self.window_slack_tokens is not None else num_tokens
-                need = min(need, (self._reach(group.spec) + slack + group.page_tokens - 1) // group.page_tokens + 2)
+                need = min(need, (self._reach(group.spec) + slack + group.page_tokens - 1) // group.page_tokens + 2
+                           + self._kept_pages(group.spec, group.page_tokens))
             if need > group.num_pages:
                 return False
         return True
 
     def _first_live_page(self, group: CacheGroup, length: int) -> int:
-        """Index of the first page that a query at position >= length may still read."""
+        """Index of the first page that a query at position >= length may still read (kept first pages aside)."""
         first_key = 0
         if group.spec.window is not None:
             first_key = max(0, length - group.spec.window + 1)
@@ -233,10 +240,11 @@ class CacheManager:
         for g, group in enumerate(self.groups):
             first = self._first_live_page(group, new_length)
             table = req.tables[g]
-            passed = [p for p in table[:first] if p != NO_PAGE]
+            kept = self._kept_pages(group.spec, group.page_tokens)
+            passed = [p for p in table[kept:first] if p != NO_PAGE]
             if passed:
                 group.pool.give_back(passed)
-                for i in range(min(first, len(table))):
+                for i in range(kept, min(first, len(table))):
                     table[i] = NO_PAGE
                 req.version += 1
 
@@ -271,7 +279,8 @@ class CacheManager:
             for g, group in enumerate(self.groups):
                 held_tokens += sum(1 for p in r.tables[g] if p != NO_PAGE) * group.page_tokens
                 first = self._first_live_page(group, r.length) * group.page_tokens
-                used_tokens += max(0, r.length - first)
+                kept = min(first, self._kept_pages(group.spec, group.page_tokens) * group.page_tokens)
+                used_tokens += max(0, r.length - first) + min(kept, r.length)
         return {
             "free_blocks": sum(g.pool.num_free for g in self.groups),
             "allocated_blocks": sum(g.pool.num_used for g in self.groups),

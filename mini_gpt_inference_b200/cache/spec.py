@@ -29,6 +29,8 @@ class PagedKVSpec:
     # Queries read only the keys of their own block of this many positions (blocks counted from
     # position 0): the pages of blocks that are over can be given back (None: no such mask).
     block: int | None = None
+    # With a window: the first tokens of the sequence that later queries still read beside it; their pages stay.
+    keep_first: int = 0
     # A token's values are the first ``v_head_dim`` features of its key row: no value pages are kept, attention
     # reads the values out of the key pages (a latent that serves as both).
     values_in_keys: bool = False
@@ -44,6 +46,8 @@ class PagedKVSpec:
             raise ValueError("window must be positive when given")
         if self.block is not None and self.block <= 0:
             raise ValueError("block must be positive when given")
+        if self.keep_first < 0 or (self.keep_first and self.window is None):
+            raise ValueError("keep_first is a number of tokens kept beside a window")
         if self.page_tokens is not None and self.page_tokens <= 0:
             raise ValueError("page_tokens must be positive when given")
         if self.num_pages is not None and self.num_pages <= 0:

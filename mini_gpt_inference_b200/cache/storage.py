@@ -27,6 +27,7 @@ class PagedKVView:
     window: int | None
     writes: bool
     values_in_keys: bool = False   # v_pages is k_pages: a token's values are the first features of its key row
+    keep_first: int = 0            # with a window: the first tokens that every query still sees
     state: torch.Tensor | None = None   # [slot, *shape], where the layer also keeps a tensor per request
 
 
@@ -61,7 +62,7 @@ class CacheStorage:
             idx = m.groups[g].layers.index(cache_layer)
             return PagedKVView(self.k[g][idx], self.v[g][idx], g, m.groups[g].page_tokens,
                                m.groups[g].spec.window, writes, m.groups[g].spec.values_in_keys,
-                               self.state.get(cache_layer))
+                               m.groups[g].spec.keep_first, self.state.get(cache_layer))
         if cache_layer in self.state:
             return StateView(self.state[cache_layer], writes)
         return None

@@ -10,7 +10,8 @@
 // Two further masks and biases, both parameters: `block` > 0 lets a query see only the keys of its own
 // block of that many positions (lo is raised to the block's first position; blocks are counted from
 // position 0 of the sequence); `slopes` (one number per head) takes slope_h * (p - j) off the score
-// of key j.
+// of key j.  `keep_first` > 0 (beside a window or a block mask): the first keep_first keys of the sequence stay in sight;
+// they are visited first, then lo..p, as one list cut into blocks of 32.
 //
 // Any key size up to 1,024 and value size up to 512 and any number of heads and kv heads (n_head a
 // multiple of n_kv_head) are accepted.  Entries of the block table are read only for positions lo..p, so
@@ -36,7 +37,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_stride, const T*
                                const T* __restrict__ gate, int gate_stride,
                                int page_tokens, int max_pages, int window, float scale, int num_pages,
                                int n_requests, const float* __restrict__ slopes, int block, float softcap,
-                               const float* __restrict__ sinks, int v_stride) {
+                               const float* __restrict__ sinks, int v_stride, int keep_first) {
     extern __shared__ float q_smem[];                     // [WARPS][head_dim]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int token = blockIdx.x;
@@ -69,9 +70,12 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_stride, const T*
     for (int i = 0; i < MAX_DPL; ++i) acc[i] = 0.f;
     float run_max = -INFINITY, run_sum = 0.f;
 
-    for (int j0 = lo; j0 <= p; j0 += 32) {
-        const int j = j0 + lane;
-        const bool valid = j <= p;
+    const int kept = min(keep_first, lo);                  // keys in front of lo that are in sight
+    const int total = kept + p - lo + 1;
+    for (int i0 = 0; i0 < total; i0 += 32) {
+        const int i = i0 + lane;
+        const int j = i < kept ? i : lo + i - kept;
+        const bool valid = i < total;
         int row = 0;                                       // row of key j in the page storage
         float s = -INFINITY;
         if (valid) {
@@ -91,7 +95,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_stride, const T*
         run_max = new_max;
 #pragma unroll
         for (int i = 0; i < MAX_DPL; ++i) acc[i] *= corr;
-        const int count = min(32, p - j0 + 1);
+        const int count = min(32, total - i0);
         for (int jj = 0; jj < count; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, prob, jj);
             const int rj = __shfl_sync(0xffffffffu, row, jj);
@@ -138,7 +142,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_stride, const T*
 // before the slopes and the softmax.  sinks: [n_head] 32-bit or null: exp(sink_h) is added to the softmax's
 // denominator of head h (no key, no value; neither scaled nor capped).  v_stride: elements between the value
 // rows of neighbouring tokens in `v_pages` (0: v_dim; larger where a token's values are the first v_dim
-// features of a wider row, its key row for instance).
+// features of a wider row, its key row for instance).  keep_first: keys at the sequence's start that stay in sight.
 // num_pages: pages of the pool (with n_requests, what guarded builds hold the indices against).
 MG_API int mg_paged_attention_general(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                                       const int* block_table, const int* token_request,
@@ -147,8 +151,9 @@ MG_API int mg_paged_attention_general(const void* q, int q_stride, const void* k
                                       int page_tokens, int max_pages,
                                       int window, float scale, int num_pages, int n_requests, int is_bf16,
                                       const float* slopes, int key_block, float softcap, const float* sinks,
-                                      int v_stride, void* stream) {
+                                      int v_stride, int keep_first, void* stream) {
     if (n_tokens == 0) return MG_OK;
+    MG_REQUIRE(keep_first >= 0, "attention: a negative number of kept keys");
     if (v_stride <= 0) v_stride = v_dim;
     MG_REQUIRE(v_stride >= v_dim && softcap >= 0.f, "attention: bad value stride or cap");
     MG_REQUIRE(n_tokens > 0 && n_head > 0 && n_kv_head > 0 && page_tokens > 0 && max_pages > 0 && key_block >= 0,
@@ -166,7 +171,7 @@ MG_API int mg_paged_attention_general(const void* q, int q_stride, const void* k
     paged_attention_generic_kernel<T, DPL><<<grid, block, smem, s>>>(                                                   \
         (const T*)q, q_stride, (const T*)k_pages, (const T*)v_pages, block_table, token_request, positions, (T*)out,    \
         n_tokens, n_head, n_kv_head, head_dim, v_dim, (const T*)gate, gate_stride, page_tokens, max_pages, window,      \
-        scale, num_pages, n_requests, slopes, key_block, softcap, sinks, v_stride)
+        scale, num_pages, n_requests, slopes, key_block, softcap, sinks, v_stride, keep_first)
     if (is_bf16) {
         if (v_dim <= 256) MG_LAUNCH_GENERIC(bf16, 8); else MG_LAUNCH_GENERIC(bf16, 16);
     } else {
@@ -188,5 +193,5 @@ MG_API int mg_paged_attention_generic(const void* qkv, const void* k_pages, cons
     return mg_paged_attention_general(qkv, (n_head + 2 * n_kv_head) * head_dim, k_pages, v_pages, block_table,
                                       token_request, positions, out, n_tokens, n_head, n_kv_head, head_dim, head_dim,
                                       nullptr, 0, page_tokens, max_pages, window, scale, num_pages, n_requests, is_bf16,
-                                      nullptr, 0, 0.f, nullptr, 0, stream);
+                                      nullptr, 0, 0.f, nullptr, 0, 0, stream);
 }

@@ -20,8 +20,10 @@
 //
 // Further, all parameters: `softcap` (a score s, scale included, becomes softcap * tanh(s / softcap)), `sinks`
 // (one learned number per head whose exponential joins the softmax's denominator, with no key and no value: it is
-// added where a row's sum is final, in the tiles' epilogue and in the merge of the ranges), and `v_stride` (a
-// token's values are the first dv features of a wider row, its key row for instance).
+// added where a row's sum is final, in the tiles' epilogue and in the merge of the ranges), `v_stride` (a
+// token's values are the first dv features of a wider row, its key row for instance), and `keep_first` (beside a
+// window: the first keep_first keys of the sequence stay in sight.  The key blocks that hold them and lie in front of
+// the window's first block are walked first; ranges are cut from the list of all these blocks).
 //
 // Keys are always read from the pages, whichever step wrote them.  Rows of pages beyond a request's
 // last key are never multiplied into a result (their values are replaced by zeros in shared memory).
@@ -62,6 +64,7 @@ struct AttnParams {
     float cap_log2;               // > 0: softcap * log2(e)
     const float* sinks;           // [H] or null
     int v_stride;                 // elements between the value rows of neighbouring tokens
+    int keep_first;               // keys at the sequence's start that every query sees
 };
 
 // What a head's sink adds to a row's sum that is held relative to the maximum m (in powers of two).
@@ -75,6 +78,16 @@ __device__ __forceinline__ int first_visible(const AttnParams& p, int pos) {
     if (p.block > 0) lo = max(lo, pos / p.block * p.block);
     return lo;
 }
+
+// The key blocks a query list walks whose first own key is `lo`: `kept` keys (whole blocks) from the sequence's start
+// that lie in front of the block which holds lo, then the keys from that block (`begin`) on.
+struct KeyWalk {
+    int kept, begin;
+    __device__ __forceinline__ KeyWalk(const AttnParams& p, int lo)
+        : kept(min((p.keep_first + KB - 1) / KB * KB, lo / KB * KB)), begin(lo / KB * KB) {}
+    __device__ __forceinline__ int key(int v) const { return v < kept ? v : begin + v - kept; }       // v-th key walked
+    __device__ __forceinline__ int last(int position) const { return kept + position - begin; }      // its place in the walk
+};
 
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -97,8 +110,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // Keys j0 .. j0+63 of one request and key/value head into shared memory, asynchronously: rows
-// [KB][DP+PAD] and [KB][DVP+PAD].  Rows outside lo..hi become zeros (they may hold anything in the
-// pages).  The caller commits the group and waits for it.
+// [KB][DP+PAD] and [KB][DVP+PAD].  Rows outside lo..hi and the kept first keys become zeros (they may hold
+// anything in the pages, or have none).  The caller commits the group and waits for it.
 __device__ __forceinline__ void cp_async16(bf16* dst, const bf16* src, bool real) {
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
     const int bytes = real ? 16 : 0;                       // 0: nothing is read, the 16 bytes become zeros
@@ -120,7 +133,7 @@ __device__ __forceinline__ void load_block(const AttnParams& p, const int* table
     for (int key = warp * 16 + (lane >> lane_shift); key < warp * 16 + 16; key += 32 >> lane_shift) {
         if (c >= chunks) continue;
         const int j = j0 + key;
-        const bool real = j >= lo && j <= hi;
+        const bool real = j <= hi && (j >= lo || j < p.keep_first);
         size_t row = 0;
         if (real) {
             const int index = page_shift >= 0 ? j >> page_shift : j / p.page_tokens;
@@ -160,12 +173,12 @@ __device__ __forceinline__ void load_q(uint32_t (&qf)[DP / 16][4], const bf16* q
 
 // One warp, its 16 rows, NT * 8 keys of the block in shared memory starting at key `k_first`:
 // scores, masks, the running maximum and sum, and O += P V.  pos/lo: the two rows' own last and first
-// visible key (pos < 0: a row without a token).
+// visible key (pos < 0: a row without a token); keys below `keep` are visible too.
 template <int DP, int DVP, int NT>
 __device__ __forceinline__ void attend(const uint32_t (&qf)[DP / 16][4], const bf16* ks, const bf16* vs, int k_first,
                                        int j_first, const int (&pos)[2], const int (&lo)[2], bool all_visible,
                                        float scale_log2, float (&m)[2], float (&l)[2], float (&o)[DVP / 8][4], int lane,
-                                       const float (&slope_log2)[2], bool biased, float cap_log2) {
+                                       const float (&slope_log2)[2], bool biased, float cap_log2, int keep) {
     float s[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
@@ -198,7 +211,7 @@ __device__ __forceinline__ void attend(const uint32_t (&qf)[DP / 16][4], const b
                 const int j = j_first + n * 8 + 2 * (lane & 3) + (e & 1), r = e >> 1;
                 float sc = s[n][e] * scale_log2;
                 if (cap_log2 > 0.f) sc = cap_log2 * tanhf(sc / cap_log2);
-                const float v = (j <= pos[r] && j >= lo[r]) ? sc - slope_log2[r] * (float)(pos[r] - j) : -INFINITY;
+                const float v = (j <= pos[r] && (j >= lo[r] || j < keep)) ? sc - slope_log2[r] * (float)(pos[r] - j) : -INFINITY;
                 s[n][e] = v;
                 bm[r] = fmaxf(bm[r], v);
             }
@@ -208,7 +221,7 @@ __device__ __forceinline__ void attend(const uint32_t (&qf)[DP / 16][4], const b
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int j = j_first + n * 8 + 2 * (lane & 3) + (e & 1), r = e >> 1;
-                const float v = (j <= pos[r] && j >= lo[r]) ? s[n][e] * scale_log2 : -INFINITY;
+                const float v = (j <= pos[r] && (j >= lo[r] || j < keep)) ? s[n][e] * scale_log2 : -INFINITY;
                 s[n][e] = v;
                 bm[r] = fmaxf(bm[r], v);
             }
@@ -324,14 +337,16 @@ attention_tiles_kernel(const AttnParams p) {
     const int warp_max_lo = warp_hi >= 0 ? first_visible(p, warp_hi) : 0;
 
     // two buffers take turns: the next block's copies are in flight while this one is multiplied
-    const int j_begin = (lo_tile / KB) * KB;
+    const KeyWalk walk(p, lo_tile);
+    const int v_last = walk.last(hi);
     const int page_shift = (p.page_tokens & (p.page_tokens - 1)) == 0 ? __ffs(p.page_tokens) - 1 : -1;
-    load_block<DP, DVP>(p, table, kv_head, j_begin, lo_tile, hi, ks, vs, warp, lane, page_shift);
+    load_block<DP, DVP>(p, table, kv_head, walk.key(0), lo_tile, hi, ks, vs, warp, lane, page_shift);
     cp_async_commit();
     int buf = 0;
-    for (int j0 = j_begin; j0 <= hi; j0 += KB, buf ^= 1) {
-        if (j0 + KB <= hi) {
-            load_block<DP, DVP>(p, table, kv_head, j0 + KB, lo_tile, hi, ks + (buf ^ 1) * STAGE, vs + (buf ^ 1) * STAGE, warp, lane,
+    for (int v = 0; v <= v_last; v += KB, buf ^= 1) {
+        const int j0 = walk.key(v);
+        if (v + KB <= v_last) {
+            load_block<DP, DVP>(p, table, kv_head, walk.key(v + KB), lo_tile, hi, ks + (buf ^ 1) * STAGE, vs + (buf ^ 1) * STAGE, warp, lane,
                                 page_shift);
             cp_async_commit();
             cp_async_wait<1>();
@@ -341,8 +356,8 @@ attention_tiles_kernel(const AttnParams p) {
         __syncthreads();
         if (j0 <= warp_hi)
             attend<DP, DVP, 8>(qf, ks + buf * STAGE, vs + buf * STAGE, 0, j0, pos, lo,
-                               j0 + KB - 1 <= warp_first_pos && j0 >= warp_max_lo, p.scale_log2, m, l, o, lane, slope_log2,
-                               biased, p.cap_log2);
+                               j0 + KB - 1 <= warp_first_pos && (j0 >= warp_max_lo || j0 + KB <= p.keep_first), p.scale_log2, m, l,
+                               o, lane, slope_log2, biased, p.cap_log2, p.keep_first);
         __syncthreads();                                    // the buffer is free for the block after the next
     }
 #pragma unroll
@@ -386,11 +401,12 @@ attention_split_kernel(const AttnParams p) {
     const bool padding = position < 0;
     if (!padding && !MG_GUARDED(attention_mma, MG_GUARD_POSITION, position, (long long)p.max_pages * p.page_tokens)) position = 0;
     const int lo_row = padding ? 0 : first_visible(p, position);
-    const int first = (lo_row / KB) * KB + split * p.split_keys;         // ranges start at the window's block
-    const int last = min(position, first + p.split_keys - 1);
+    const KeyWalk walk(p, lo_row);
+    const int first = split * p.split_keys;                  // ranges are cut from the walk, which starts at a block
+    const int last = min(walk.last(position), first + p.split_keys - 1);
     // ranges that hold keys of this token; the others have nothing to do (the grid is sized for the
     // longest context there can be)
-    const int live = padding ? 0 : (position - (lo_row / KB) * KB) / p.split_keys + 1;
+    const int live = padding ? 0 : walk.last(position) / p.split_keys + 1;
     if (split >= live) {
         if (padding && split == 0)                                        // a padding row's output is zeros
             for (int i = tid; i < group * p.dv; i += 128)
@@ -421,12 +437,13 @@ attention_split_kernel(const AttnParams p) {
         uint32_t qf[DP / 16][4];
         load_q<DP>(qf, qrow[0], qrow[1], p.d, lane);
         const int page_shift = (p.page_tokens & (p.page_tokens - 1)) == 0 ? __ffs(p.page_tokens) - 1 : -1;
-        load_block<DP, DVP>(p, table, kv_head, first, lo_row, last, ks, vs, warp, lane, page_shift);
+        load_block<DP, DVP>(p, table, kv_head, walk.key(first), lo_row, position, ks, vs, warp, lane, page_shift);
         cp_async_commit();
         int buf = 0;
-        for (int j0 = first; j0 <= last; j0 += KB, buf ^= 1) {
-            if (j0 + KB <= last) {
-                load_block<DP, DVP>(p, table, kv_head, j0 + KB, lo_row, last, ks + (buf ^ 1) * STAGE, vs + (buf ^ 1) * STAGE, warp,
+        for (int v = first; v <= last; v += KB, buf ^= 1) {
+            const int j0 = walk.key(v);
+            if (v + KB <= last) {
+                load_block<DP, DVP>(p, table, kv_head, walk.key(v + KB), lo_row, position, ks + (buf ^ 1) * STAGE, vs + (buf ^ 1) * STAGE, warp,
                                     lane, page_shift);
                 cp_async_commit();
                 cp_async_wait<1>();
@@ -434,9 +451,9 @@ attention_split_kernel(const AttnParams p) {
                 cp_async_wait<0>();
             }
             __syncthreads();
-            if (j0 + warp * 16 <= last)
+            if (j0 + warp * 16 <= position)
                 attend<DP, DVP, 2>(qf, ks + buf * STAGE, vs + buf * STAGE, warp * 16, j0 + warp * 16, pos, lo, false,
-                                   p.scale_log2, m, l, o, lane, slope_log2, biased, p.cap_log2);
+                                   p.scale_log2, m, l, o, lane, slope_log2, biased, p.cap_log2, p.keep_first);
             __syncthreads();
         }
     }
@@ -531,8 +548,8 @@ __global__ void attention_merge_kernel(const AttnParams p) {
         for (int c = threadIdx.x; c < p.dv; c += blockDim.x) orow[c] = __float2bfloat16_rn(0.f);
         return;
     }
-    const int lo_row = first_visible(p, position);
-    const int live = min(min(p.splits, MERGE_MAX), (position - (lo_row / KB) * KB) / p.split_keys + 1);   // ranges that hold keys
+    const int live = min(min(p.splits, MERGE_MAX),
+                         KeyWalk(p, first_visible(p, position)).last(position) / p.split_keys + 1);   // ranges that hold keys
     for (int s = threadIdx.x; s < live; s += blockDim.x) weight[s] = p.part_ml[(base + s) * 2];
     __syncthreads();
     if (threadIdx.x < 32) {
@@ -872,7 +889,8 @@ MG_API long long mg_attention_mma_scratch_floats(int n_tokens, int n_head, int d
 // scratch of mg_attention_mma_scratch_floats floats; counters: n_tokens * n_kv_head zeros that are left
 // as zeros, or null to merge the ranges in a second kernel); 0: n_tiles tiles of tile_tokens tokens, found
 // from req_q_start / req_q_len.  slopes: [n_head] 32-bit or null; key_block <= 0: no block mask; softcap <= 0: none;
-// sinks: [n_head] 32-bit or null; v_stride: elements between value rows (0: dv).  Returns MG_ERR_UNSUPPORTED for sizes
+// sinks: [n_head] 32-bit or null; v_stride: elements between value rows (0: dv); keep_first: keys at the sequence's
+// start that stay in sight beside a window.  Returns MG_ERR_UNSUPPORTED for sizes
 // it does not take.
 MG_API int mg_attention_mma(const void* q, int q_stride, const void* k_pages, const void* v_pages, const int* block_table,
                             const int* token_request, const int* positions, const int* req_q_start,
@@ -880,8 +898,9 @@ MG_API int mg_attention_mma(const void* q, int q_stride, const void* k_pages, co
                             int* counters, int n_tokens, int n_requests, int n_head, int n_kv_head, int d, int dv, int page_tokens,
                             int max_pages, int window, float scale, int num_pages, int single_tokens, int n_tiles,
                             int tile_tokens, int splits, int split_keys, const float* slopes, int key_block, float softcap,
-                            const float* sinks, int v_stride, void* stream) {
+                            const float* sinks, int v_stride, int keep_first, void* stream) {
     if (n_tokens == 0) return MG_OK;
+    MG_REQUIRE(keep_first >= 0, "attention: a negative number of kept keys");
     MG_REQUIRE(n_tokens > 0 && n_head > 0 && n_kv_head > 0 && n_head % n_kv_head == 0 && page_tokens > 0 && max_pages > 0,
                "attention: bad sizes");
     const int group = n_head / n_kv_head;
@@ -900,7 +919,7 @@ MG_API int mg_attention_mma(const void* q, int q_stride, const void* k_pages, co
     p.page_tokens = page_tokens; p.max_pages = max_pages; p.window = window > 0 ? window : 0; p.num_pages = num_pages;
     p.tile_tokens = tile_tokens; p.splits = splits; p.split_keys = split_keys; p.scale_log2 = scale * LOG2E;
     p.slopes = slopes; p.block = key_block > 0 ? key_block : 0;
-    p.cap_log2 = softcap > 0.f ? softcap * LOG2E : 0.f; p.sinks = sinks; p.v_stride = v_stride;
+    p.cap_log2 = softcap > 0.f ? softcap * LOG2E : 0.f; p.sinks = sinks; p.v_stride = v_stride; p.keep_first = keep_first;
     if (single_tokens) {
         MG_REQUIRE(scratch != nullptr && splits > 0 && splits <= 65535 && split_keys > 0 && split_keys % KB == 0,
                    "attention: the ranges of keys want scratch and sizes that are multiples of %d", KB);
@@ -954,7 +973,7 @@ MG_API int mg_attention_wide(const void* q, int q_stride, const void* k_pages, c
     p.page_tokens = page_tokens; p.max_pages = max_pages; p.window = window > 0 ? window : 0; p.num_pages = num_pages;
     p.tile_tokens = 0; p.splits = splits; p.split_keys = split_keys; p.scale_log2 = scale * LOG2E;
     p.slopes = nullptr; p.block = 0;
-    p.cap_log2 = softcap > 0.f ? softcap * LOG2E : 0.f; p.sinks = sinks; p.v_stride = d;
+    p.cap_log2 = softcap > 0.f ? softcap * LOG2E : 0.f; p.sinks = sinks; p.v_stride = d; p.keep_first = 0;
     if (single_tokens) {
         MG_REQUIRE(scratch != nullptr && splits > 0 && splits <= 65535 && split_keys > 0 && split_keys % KB == 0,
                    "attention: the ranges of keys want scratch and sizes that are multiples of %d", KB);

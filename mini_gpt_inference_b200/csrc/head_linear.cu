@@ -3,7 +3,7 @@
 //   out[n, h, j] = sum_i x[n, h, i] * W_h[j, i]      (rows_are_inputs = 0: W is [H * J, I], a head's rows are its outputs)
 //   out[n, h, j] = sum_i x[n, h, i] * W_h[i, j]      (rows_are_inputs = 1: W is [H * I, J], a head's rows are its inputs)
 //
-// optionally times the logistic function of a gate value per output.  An attention whose keys and values are
+// optionally times the logistic function of a gate value per output, or of one that a head's outputs share.  An attention whose keys and values are
 // made from a small latent per token uses both forms: queries are carried into the latent's space with the
 // transposed key matrix of their head (so that scores are taken against the cached latents themselves), and the
 // heads' weighted latents are carried to value space with the value matrix of their head.
@@ -20,7 +20,7 @@ constexpr int TOK = 32, OUT = 64, KC = 32, THREADS = 256;
 template <typename T>
 __global__ void __launch_bounds__(THREADS)
 head_linear_kernel(const T* __restrict__ x, int x_ld, int x_off, int x_head, const T* __restrict__ w, int rows_are_inputs,
-                   const T* __restrict__ gate, int gate_ld, T* __restrict__ out, int out_ld, int out_off, int out_head,
+                   const T* __restrict__ gate, int gate_ld, int head_gate, T* __restrict__ out, int out_ld, int out_off, int out_head,
                    int n_tokens, int I, int J) {
     __shared__ float xs[TOK][KC + 1];
     __shared__ float ws[KC][OUT + 1];
@@ -66,7 +66,7 @@ head_linear_kernel(const T* __restrict__ x, int x_ld, int x_off, int x_head, con
         const int n = n0 + tg * (TOK / 4) + u;
         if (n >= n_tokens) continue;
         float v = acc[u];
-        if (gate) v *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)n * gate_ld + (size_t)h * J + j0 + jl])));
+        if (gate) v *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)n * gate_ld + (head_gate ? h : (size_t)h * J + j0 + jl)])));
         out[(size_t)n * out_ld + out_off + (size_t)h * out_head + j0 + jl] = from_float<T>(v);
     }
 }
@@ -98,7 +98,7 @@ __device__ __forceinline__ void hl_ldsm_t(uint32_t (&r)[4], const bf16* p) {
 template <int MN>            // outputs per CTA: 64, or 16 for steps of few tokens (more CTAs share the heads' matrices)
 __global__ void __launch_bounds__(128)
 head_linear_mma_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_head, const bf16* __restrict__ w,
-                       int rows_are_inputs, const bf16* __restrict__ gate, int gate_ld, bf16* __restrict__ out, int out_ld,
+                       int rows_are_inputs, const bf16* __restrict__ gate, int gate_ld, int head_gate, bf16* __restrict__ out, int out_ld,
                        int out_off, int out_head, int n_tokens, int I, int J) {
     __shared__ __align__(16) bf16 xs[MT][MK + MPAD];
     __shared__ __align__(16) bf16 ws[64][64 + MPAD];       // [j][i], or [i][j] if the rows are inputs
@@ -154,12 +154,16 @@ head_linear_mma_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_he
     for (int r = 0; r < 4; ++r) {
         const int n = n0 + warp * 32 + (lane >> 2) + 8 * r;
         if (n >= n_tokens) continue;
+        const float shared = head_gate ? 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)n * gate_ld + h]))) : 1.f;
 #pragma unroll
         for (int t = 0; t < MN / 8; ++t) {
             const int j = j0 + t * 8 + 2 * (lane & 3);
             if (j >= J) continue;
             float a = acc[r >> 1][t][2 * (r & 1)], b = acc[r >> 1][t][2 * (r & 1) + 1];
-            if (gate) {
+            if (head_gate) {
+                a *= shared;
+                b *= shared;
+            } else if (gate) {
                 const __nv_bfloat162 g = *reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)n * gate_ld + (size_t)h * J + j);
                 a *= 1.0f / (1.0f + expf(-__bfloat162float(g.x)));
                 b *= 1.0f / (1.0f + expf(-__bfloat162float(g.y)));
@@ -187,7 +191,7 @@ __device__ __forceinline__ void hl_copy16(bf16* dst, const bf16* src, bool real)
 
 __global__ void __launch_bounds__(128)
 head_linear_few_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_head, const bf16* __restrict__ w,
-                       int rows_are_inputs, const bf16* __restrict__ gate, int gate_ld, bf16* __restrict__ out, int out_ld,
+                       int rows_are_inputs, const bf16* __restrict__ gate, int gate_ld, int head_gate, bf16* __restrict__ out, int out_ld,
                        int out_off, int out_head, int n_tokens, int I, int J) {
     extern __shared__ __align__(16) uint8_t few_raw[];
     __shared__ float part[4][FEW][FEW_OUT];
@@ -246,7 +250,11 @@ head_linear_few_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_he
         float v[2];
 #pragma unroll
         for (int u = 0; u < 2; ++u) v[u] = (part[0][n][c + u] + part[1][n][c + u]) + (part[2][n][c + u] + part[3][n][c + u]);
-        if (gate) {
+        if (head_gate) {
+            const float shared = 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)n * gate_ld + h])));
+            v[0] *= shared;
+            v[1] *= shared;
+        } else if (gate) {
             const __nv_bfloat162 g = *reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)n * gate_ld + (size_t)h * J + j);
             v[0] *= 1.0f / (1.0f + expf(-__bfloat162float(g.x)));
             v[1] *= 1.0f / (1.0f + expf(-__bfloat162float(g.y)));
@@ -258,23 +266,24 @@ head_linear_few_kernel(const bf16* __restrict__ x, int x_ld, int x_off, int x_he
 }  // namespace
 
 // x: rows of x_ld elements, head h's I inputs from column x_off + h * x_head; w: [n_head * J, I] or, if
-// rows_are_inputs, [n_head * I, J]; gate: rows of gate_ld elements whose first n_head * J are gate values, or
-// null; out: rows of out_ld elements, head h's J outputs from column out_off + h * out_head.
+// rows_are_inputs, [n_head * I, J]; gate: rows of gate_ld elements whose first n_head * J (head_gate: n_head, one
+// per head) are gate values, or null; out: rows of out_ld elements, head h's J outputs from column out_off + h * out_head.
 MG_API int mg_head_linear(const void* x, int x_ld, int x_off, int x_head, const void* w, int rows_are_inputs,
-                          const void* gate, int gate_ld, void* out, int out_ld, int out_off, int out_head, int n_tokens,
+                          const void* gate, int gate_ld, int head_gate, void* out, int out_ld, int out_off, int out_head, int n_tokens,
                           int n_head, int I, int J, int is_bf16, void* stream) {
     if (n_tokens == 0) return MG_OK;
     MG_REQUIRE(n_tokens > 0 && n_head > 0 && I > 0 && J > 0, "head_linear: bad sizes");
+    if (gate == nullptr) head_gate = 0;
     MG_REQUIRE(x_off >= 0 && x_head >= I && x_off + (long long)(n_head - 1) * x_head + I <= x_ld &&
                    out_off >= 0 && out_head >= J && out_off + (long long)(n_head - 1) * out_head + J <= out_ld &&
-                   (gate == nullptr || gate_ld >= n_head * J),
+                   (gate == nullptr || gate_ld >= (head_gate ? n_head : n_head * J)),
                "head_linear: heads outside the rows");
     const dim3 grid(ceil_div(n_tokens, TOK), n_head, ceil_div(J, OUT)), block(THREADS);
     MG_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "head_linear: too many heads or outputs");
     cudaStream_t s = (cudaStream_t)stream;
     const bool vectors = I % 8 == 0 && J % 8 == 0 && x_ld % 8 == 0 && x_off % 8 == 0 && x_head % 8 == 0 && out_ld % 2 == 0 &&
-                         out_off % 2 == 0 && out_head % 2 == 0 && gate_ld % 2 == 0 && (uintptr_t)x % 16 == 0 &&
-                         (uintptr_t)w % 16 == 0 && (uintptr_t)out % 4 == 0 && (uintptr_t)gate % 4 == 0;
+                         out_off % 2 == 0 && out_head % 2 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+                         (uintptr_t)out % 4 == 0 && (head_gate || (gate_ld % 2 == 0 && (uintptr_t)gate % 4 == 0));
     if (is_bf16 && vectors && n_tokens <= FEW && few_smem(I, rows_are_inputs) <= 96 * 1024) {
         static bool configured = false;
         if (!configured) {
@@ -285,7 +294,7 @@ MG_API int mg_head_linear(const void* x, int x_ld, int x_off, int x_head, const 
         MG_REQUIRE(ceil_div(J, FEW_OUT) <= 65535, "head_linear: too many outputs");
         const cudaError_t ef = mg_launch(head_linear_few_kernel, dim3(n_head, ceil_div(J, FEW_OUT)), dim3(128),
                                          few_smem(I, rows_are_inputs), s, true, (const bf16*)x, x_ld, x_off, x_head, (const bf16*)w,
-                                         rows_are_inputs, (const bf16*)gate, gate_ld, (bf16*)out, out_ld, out_off, out_head,
+                                         rows_are_inputs, (const bf16*)gate, gate_ld, head_gate, (bf16*)out, out_ld, out_off, out_head,
                                          n_tokens, I, J);
         if (ef != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "head_linear (few tokens): %s", cudaGetErrorString(ef));
         return MG_OK;
@@ -296,20 +305,20 @@ MG_API int mg_head_linear(const void* x, int x_ld, int x_off, int x_head, const 
         MG_REQUIRE(tiles.z <= 65535, "head_linear: too many outputs");
         const cudaError_t em =
             mn == 16 ? mg_launch(head_linear_mma_kernel<16>, tiles, dim3(128), 0, s, true, (const bf16*)x, x_ld, x_off, x_head,
-                                 (const bf16*)w, rows_are_inputs, (const bf16*)gate, gate_ld, (bf16*)out, out_ld, out_off, out_head,
+                                 (const bf16*)w, rows_are_inputs, (const bf16*)gate, gate_ld, head_gate, (bf16*)out, out_ld, out_off, out_head,
                                  n_tokens, I, J)
                      : mg_launch(head_linear_mma_kernel<64>, tiles, dim3(128), 0, s, true, (const bf16*)x, x_ld, x_off, x_head,
-                                 (const bf16*)w, rows_are_inputs, (const bf16*)gate, gate_ld, (bf16*)out, out_ld, out_off, out_head,
+                                 (const bf16*)w, rows_are_inputs, (const bf16*)gate, gate_ld, head_gate, (bf16*)out, out_ld, out_off, out_head,
                                  n_tokens, I, J);
         if (em != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "head_linear (mma): %s", cudaGetErrorString(em));
         return MG_OK;
     }
     const cudaError_t e =
         is_bf16 ? mg_launch(head_linear_kernel<bf16>, grid, block, 0, s, true, (const bf16*)x, x_ld, x_off, x_head,
-                            (const bf16*)w, rows_are_inputs, (const bf16*)gate, gate_ld, (bf16*)out, out_ld, out_off,
+                            (const bf16*)w, rows_are_inputs, (const bf16*)gate, gate_ld, head_gate, (bf16*)out, out_ld, out_off,
                             out_head, n_tokens, I, J)
                 : mg_launch(head_linear_kernel<float>, grid, block, 0, s, true, (const float*)x, x_ld, x_off, x_head,
-                            (const float*)w, rows_are_inputs, (const float*)gate, gate_ld, (float*)out, out_ld, out_off,
+                            (const float*)w, rows_are_inputs, (const float*)gate, gate_ld, head_gate, (float*)out, out_ld, out_off,
                             out_head, n_tokens, I, J);
     if (e != cudaSuccess) return mg_set_error(MG_ERR_CUDA, "head_linear: %s", cudaGetErrorString(e));
     return MG_OK;

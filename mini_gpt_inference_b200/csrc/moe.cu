@@ -2,12 +2,13 @@
 // matrix products over the groups, and the weighted sum back into the residual stream.
 //
 //   route:   z = W_r h (32-bit), the `top` largest z choose experts (ties: the lower index), their
-//            weights are softmax over the chosen z alone; optionally g = sigmoid(w_g . h), one number
+//            weights are softmax over the chosen z alone (or each one's own logistic function); optionally g = sigmoid(w_g . h), one number
 //            per token (the gate of an expert that every token uses; such experts can join the chosen ones as
 //            further entries of every token, g their weight).
 //   group:   entry (token, k) -> a slot; the slots of one expert are contiguous and in entry order.
 //   experts: H[slot] = silu(W_gate[e] h) * (W_up[e] h), or act(W_up[e] h) for experts without a gate;
-//            Y[slot] = weight[slot] * W_down[e] H[slot]  (32-bit)
+//            Y[slot] = weight[slot] * W_down[e] H[slot]  (32-bit).  A weight that belongs on the experts' inputs
+//            multiplies the first product's sums instead (W (w h) = w (W h))
 //   combine: x[token] += sum_k Y[slot of (token, k)], k in order: the same sum whatever the grouping.
 //
 // Nothing here depends on the host knowing how many tokens an expert got: grids are sized for the
@@ -77,7 +78,7 @@ template <typename T, int NT, int WARPS>
 __global__ void __launch_bounds__(32 * WARPS)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ w_gate,
                  const int* __restrict__ positions, int* __restrict__ ids, float* __restrict__ weights,
-                 float* __restrict__ gate, int n_tokens, int width, int n_experts, int top, int always) {
+                 float* __restrict__ gate, int n_tokens, int width, int n_experts, int top, int always, int scoring, float scale) {
     extern __shared__ float z_all[];                       // per token: [n_experts], then the gate
     pdl_trigger();
     pdl_wait();
@@ -91,7 +92,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
         if (lane == 0)
 #pragma unroll
             for (int u = 0; u < NT; ++u)
-                z_all[u * (n_experts + 1) + e] = e < n_experts ? dot[u] : 1.0f / (1.0f + expf(-dot[u]));
+                z_all[u * (n_experts + 1) + e] = e < n_experts && !scoring ? dot[u] : 1.0f / (1.0f + expf(-dot[u]));
     }
     __syncthreads();
     const int token = first + warp;
@@ -126,7 +127,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
         }
         if (best_e >= n_experts) best_e = k;               // logits that are not numbers: still a valid choice
         if (k == 0) z_max = best;
-        const float p = expf(best - z_max);
+        const float p = scoring ? best * scale : expf(best - z_max);
         sum += p;
         if (lane == 0) {
             ids[k] = best_e;
@@ -135,7 +136,8 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
         }
         __syncwarp();
     }
-    const float inv = 1.0f / sum;
+    if (scoring) return;
+    const float inv = scale / sum;
     for (int k = lane; k < top; k += 32) weights[k] *= inv;
 }
 
@@ -334,9 +336,10 @@ __device__ __forceinline__ float gated_value(int act, float limit, float g, floa
 // A unit without a gate: its one hidden feature z, by `act` (0: max(z, 0)^2, 1: gelu_tanh(z), 2: silu(z)).
 __device__ __forceinline__ float plain_value(int act, float z) { return act == 0 ? relu_sq(z) : act == 1 ? gelu_tanh(z) : silu(z); }
 
-// FORM 1 (gated): out[slot, n] = silu(a . w[e][n]) * (a . w[e][inner + n]),  a = x[token of slot]   (T out)
-// FORM 2 (plain): out[slot, n] = act(a . w[e][n]),                           a = x[token of slot]   (T out)
-// FORM 0 (out):   out[slot, n] = scale[entry of slot] * (a . w[e][n]),       a = x[slot]            (32-bit out)
+// With s = scale[entry of slot], or 1 where scale is null:
+// FORM 1 (gated): out[slot, n] = silu(s (a . w[e][n])) * s (a . w[e][inner + n]),  a = x[token of slot]   (T out)
+// FORM 2 (plain): out[slot, n] = act(s (a . w[e][n])),                             a = x[token of slot]   (T out)
+// FORM 0 (out):   out[slot, n] = s (a . w[e][n]),                                  a = x[slot]            (32-bit out)
 template <typename T, int FORM>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, long long w_expert_stride,
@@ -412,15 +415,15 @@ moe_gemm_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, long 
         const int m = m0 + tr * TM + i;
         if (m >= count) continue;
         const size_t slot = (size_t)first + m;
-        const float sc = FORM != 0 ? 1.f : scale[slot_entry[slot]];
+        const float sc = scale ? scale[slot_entry[slot]] : 1.f;
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int n = n0 + tc * TN + j;
             if (n >= N) continue;
             if constexpr (GLU)
-                reinterpret_cast<T*>(out)[slot * N + n] = from_float<T>(gated_value(act, limit, acc[i][j], acc_u[i][j]));
+                reinterpret_cast<T*>(out)[slot * N + n] = from_float<T>(gated_value(act, limit, acc[i][j] * sc, acc_u[i][j] * sc));
             else if constexpr (FORM == 2)
-                reinterpret_cast<T*>(out)[slot * N + n] = from_float<T>(plain_value(act, acc[i][j]));
+                reinterpret_cast<T*>(out)[slot * N + n] = from_float<T>(plain_value(act, acc[i][j] * sc));
             else
                 reinterpret_cast<float*>(out)[slot * N + n] = acc[i][j] * sc;
         }
@@ -574,12 +577,13 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
             const int m = m0 + m_warp + i * 16 + (lane >> 2) + 8 * half;
             if (m >= count) continue;
             const size_t slot = (size_t)first + m;
+            const float sc = scale ? scale[slot_entry[slot]] : 1.f;
             if (GLU) {
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     const int n = n0 + wc * 32 + j * 8 + 2 * (lane & 3);
-                    const float v0 = gated_value(act, limit, acc[i][j][2 * half], acc[i][j + 4][2 * half]);
-                    const float v1 = gated_value(act, limit, acc[i][j][2 * half + 1], acc[i][j + 4][2 * half + 1]);
+                    const float v0 = gated_value(act, limit, acc[i][j][2 * half] * sc, acc[i][j + 4][2 * half] * sc);
+                    const float v1 = gated_value(act, limit, acc[i][j][2 * half + 1] * sc, acc[i][j + 4][2 * half + 1] * sc);
                     bf16* o = reinterpret_cast<bf16*>(out) + slot * N + n;
                     if (n + 1 < N && (N & 1) == 0) *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, v1);
                     else {
@@ -591,7 +595,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     const int n = n0 + wc * 64 + j * 8 + 2 * (lane & 3);
-                    const float v0 = plain_value(act, acc[i][j][2 * half]), v1 = plain_value(act, acc[i][j][2 * half + 1]);
+                    const float v0 = plain_value(act, acc[i][j][2 * half] * sc), v1 = plain_value(act, acc[i][j][2 * half + 1] * sc);
                     bf16* o = reinterpret_cast<bf16*>(out) + slot * N + n;
                     if (n + 1 < N && (N & 1) == 0) *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, v1);
                     else {
@@ -600,7 +604,6 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
                     }
                 }
             } else {
-                const float sc = scale[slot_entry[slot]];
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     const int n = n0 + wc * 64 + j * 8 + 2 * (lane & 3);
@@ -653,10 +656,11 @@ __global__ void glu_kernel(const T* __restrict__ gu, const float* __restrict__ s
 // h: [n_tokens, width] (bfloat16 if is_bf16 else 32-bit); w_router: [n_experts, width] and w_gate:
 // [width] (null: no gate), 32-bit; positions: [n_tokens] or null; ids, weights: [n_tokens, top + always]: behind a
 // token's chosen experts the experts n_experts .. n_experts + always - 1, which every token uses, with the gate's value
-// (1 without a gate) as their weight; gate: [n_tokens] or null.
+// (1 without a gate) as their weight; gate: [n_tokens] or null.  scoring 1: the logistic functions of the z are compared
+// and are, times scale, the weights; 0: scale times the softmax over the chosen z.
 MG_API int mg_moe_route(const void* h, const float* w_router, const float* w_gate, const int* positions, int* ids,
                         float* weights, float* gate, int n_tokens, int width, int n_experts, int top, int always,
-                        int is_bf16, void* stream) {
+                        int scoring, float scale, int is_bf16, void* stream) {
     if (n_tokens == 0) return MG_OK;
     MG_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top > 0 && top <= n_experts, "moe route: bad sizes");
     MG_REQUIRE(gate == nullptr || w_gate != nullptr, "moe route: a gate wants its weights");
@@ -671,12 +675,12 @@ MG_API int mg_moe_route(const void* h, const float* w_router, const float* w_gat
         auto kernel = per != 1 ? moe_route_kernel<bf16, ROUTE_TOKENS, ROUTE_WARPS>
                     : warps == ROUTE_WARPS ? moe_route_kernel<bf16, 1, ROUTE_WARPS> : moe_route_kernel<bf16, 1, ROUTE_WARPS_FEW>;
         e = mg_launch(kernel, grid, block, smem, (cudaStream_t)stream, true, (const bf16*)h, w_router, w_gate, positions, ids,
-                      weights, gate, n_tokens, width, n_experts, top, always);
+                      weights, gate, n_tokens, width, n_experts, top, always, scoring, scale);
     } else {
         auto kernel = per != 1 ? moe_route_kernel<float, ROUTE_TOKENS, ROUTE_WARPS>
                     : warps == ROUTE_WARPS ? moe_route_kernel<float, 1, ROUTE_WARPS> : moe_route_kernel<float, 1, ROUTE_WARPS_FEW>;
         e = mg_launch(kernel, grid, block, smem, (cudaStream_t)stream, true, (const float*)h, w_router, w_gate, positions, ids,
-                      weights, gate, n_tokens, width, n_experts, top, always);
+                      weights, gate, n_tokens, width, n_experts, top, always, scoring, scale);
     }
     MG_LAUNCHED(e, "moe route");
     return MG_OK;
@@ -724,7 +728,8 @@ MG_API int mg_moe_group(const int* ids, int n_entries, int n_experts, int* offse
 // act, limit: what the first product's epilogue computes (gated_value, plain_value).
 // form 1 (gated): x [x_rows, ldx] gathered by token, w [n_experts, 2 N, K], out [n_entries, N] in the inputs' type.
 // form 2 (plain): the same with w [n_experts, N, K].
-// form 0 (out):   x [n_entries, ldx] by slot, w [n_experts, N, K], scale [n_entries] by entry, out [n_entries, N] 32-bit.
+// form 0 (out):   x [n_entries, ldx] by slot, w [n_experts, N, K], out [n_entries, N] 32-bit.
+// scale: [n_entries] by entry, a factor on the product (in front of the activation), or null.
 // max_rows: the most slots one expert can have (the tokens of the step).
 MG_API int mg_moe_gemm(const void* x, int ldx, const void* w, const int* offsets, const int* slot_entry, int top,
                        const float* scale, void* out, int n_experts, int max_rows, int N, int K, int x_rows, int form,
@@ -732,7 +737,6 @@ MG_API int mg_moe_gemm(const void* x, int ldx, const void* w, const int* offsets
     if (max_rows == 0) return MG_OK;
     MG_REQUIRE(n_experts > 0 && n_experts <= 65535 && max_rows > 0 && N > 0 && K > 0 && ldx >= K && top > 0 && form >= 0 && form <= 2,
                "moe gemm: bad sizes");
-    MG_REQUIRE(form != 0 || scale != nullptr, "moe gemm: the second product wants the entries' weights");
     const dim3 grid(ceil_div(N, BN), ceil_div(max_rows, BM), n_experts), block(256);
     MG_REQUIRE(grid.y <= 65535, "moe gemm: too many rows");
     const long long stride = (long long)(form == 1 ? 2 : 1) * N * K;

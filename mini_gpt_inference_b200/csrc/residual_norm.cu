@@ -5,8 +5,9 @@
 //               or the weighted sum of two sublayers that ran side by side), or the sum of the rows that a token's
 //               entries point to (experts that wrote their results apart); with `center` the mean of y is taken off
 //               first (a layer norm).  With `clear` the inputs are left as zeros: the buffer a sublayer added its output
-//               into serves the next sublayer as it is.  Optionally the new x is also written in bfloat16: what a
-//               sublayer that reads the stream itself wants next
+//               into serves the next sublayer as it is.  Optionally the new x is also written in bfloat16 (what a
+//               sublayer that reads the stream itself wants next), or an RMS norm of it, x / sqrt(mean(x^2) + eps2) *
+//               (offset2 + w2), in bfloat16 or 32-bit (what a sublayer with a norm in front of it wants next)
 // add_rows:     x += [e] + v    (e: rows like x, or none; v: one row for all tokens)
 // scaled_sum:   x += sa * a + sb * b   (with `clear`, a and b are left as zeros)
 // softcap:      x <- cap * tanh(x / cap)
@@ -42,7 +43,10 @@ struct NormOutput {
     float eps, offset, scale;      // x += scale * norm(y) * (offset + w)
     int center;                    // take the row's mean off first (a layer norm)
     int clear;                     // leave a and b as zeros
-    bf16* rows;                    // the new stream in bfloat16 as well, or null
+    bf16* rows;                    // the new stream (with w2: its norm) in bfloat16 as well, or null
+    float* rows32;                 // with w2: its norm in 32-bit, or null
+    const float* w2;               // the weights of the norm in front of what comes next, or null
+    float eps2, offset2;
 };
 
 __device__ __forceinline__ int entry_row(const NormInput& in, size_t row, int k) {
@@ -81,16 +85,26 @@ norm_add_kernel(const NormInput in, const NormOutput out, int rows, int width) {
         sq = fmaf(y, y, sq);
     }
     const float rstd = 1.0f / sqrtf(warp_sum(sq) / (float)width + out.eps);
+    float sq2 = 0.f;
     for (int c = lane; c < width; c += 32) {
         const size_t i = (size_t)row * width + c;
         const float y = norm_input(in, row, width, c) - mean;
         const float x = out.x[i] + out.scale * (y * rstd * (out.offset + out.w[c]));
         out.x[i] = x;
-        if (out.rows) out.rows[i] = __float2bfloat16_rn(x);
+        sq2 = fmaf(x, x, sq2);
+        if (out.rows && !out.w2) out.rows[i] = __float2bfloat16_rn(x);
         if (out.clear) {
             in.a[i] = 0.f;
             if (in.b) in.b[i] = 0.f;
         }
+    }
+    if (!out.w2) return;
+    const float r2 = 1.0f / sqrtf(warp_sum(sq2) / (float)width + out.eps2);
+    for (int c = lane; c < width; c += 32) {               // (a lane reads what it wrote itself)
+        const size_t i = (size_t)row * width + c;
+        const float h = out.x[i] * r2 * (out.offset2 + out.w2[c]);
+        if (out.rows) out.rows[i] = __float2bfloat16_rn(h);
+        else out.rows32[i] = h;
     }
 }
 
@@ -174,7 +188,8 @@ norm_add_vec_kernel(const NormInput in, const NormOutput out, int width) {
             const float4 r = make_float4(xv[u].x + sc * (y[u].x * rstd * (off + wv[u].x)), xv[u].y + sc * (y[u].y * rstd * (off + wv[u].y)),
                                          xv[u].z + sc * (y[u].z * rstd * (off + wv[u].z)), xv[u].w + sc * (y[u].w * rstd * (off + wv[u].w)));
             xr[i] = r;
-            if (out.rows) {
+            xv[u] = r;
+            if (out.rows && !out.w2) {
                 __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(out.rows + 4 * (base + i));
                 o[0] = __floats2bfloat162_rn(r.x, r.y);
                 o[1] = __floats2bfloat162_rn(r.z, r.w);
@@ -183,6 +198,26 @@ norm_add_vec_kernel(const NormInput in, const NormOutput out, int width) {
                 ar[i] = zero;
                 if (br) br[i] = zero;
             }
+        }
+    }
+    if (!out.w2) return;
+    const float4* w2r = reinterpret_cast<const float4*>(out.w2);
+    sq = 0.f;
+#pragma unroll
+    for (int u = 0; u < ROW_VECS; ++u) {
+        sq = fmaf(xv[u].x, xv[u].x, fmaf(xv[u].y, xv[u].y, fmaf(xv[u].z, xv[u].z, fmaf(xv[u].w, xv[u].w, sq))));
+        const int i = tid + u * ROW_THREADS;
+        if (i < vecs) wv[u] = w2r[i];
+    }
+    const float r2 = 1.0f / sqrtf(row_total(sq, red[0]) / (float)width + out.eps2), off2 = out.offset2;
+#pragma unroll
+    for (int u = 0; u < ROW_VECS; ++u) {
+        const int i = tid + u * ROW_THREADS;
+        if (i < vecs) {
+            const float a = xv[u].x * r2 * (off2 + wv[u].x), b = xv[u].y * r2 * (off2 + wv[u].y),
+                        c = xv[u].z * r2 * (off2 + wv[u].z), d = xv[u].w * r2 * (off2 + wv[u].w);
+            if (out.rows) store4(out.rows + 4 * (base + i), a, b, c, d);
+            else store4(out.rows32 + 4 * (base + i), a, b, c, d);
         }
     }
 }
@@ -254,20 +289,23 @@ __global__ void token_gate_kernel(const float* __restrict__ g, const int* __rest
 }  // namespace
 
 // x: [rows, width] 32-bit, in place; a (and b, or null): [rows, width] 32-bit (zeroed if clear); w: [width] 32-bit.
-// center: the row's mean is taken off first.  scale: factor on what is added.  out_rows: [rows, width] bfloat16 or null.
+// center: the row's mean is taken off first.  scale: factor on what is added.  out_rows: [rows, width] bfloat16 (32-bit
+// if rows_32bit, only with w2) or null; w2 ([width] 32-bit or null), eps2, offset2: the norm that out_rows is of the new x.
 // entry_slot (or null): [rows, top] rows of a, [n_slots, width], whose sum is the input (below zero: none); then b must be
 // null and clear 0.
 MG_API int mg_norm_add(float* x, float* a, float sa, float* b, float sb, const int* entry_slot, int top, int n_slots,
                        const float* w, int rows, int width, float eps, float offset, int center, float scale, int clear,
-                       void* out_rows, void* stream) {
+                       void* out_rows, int rows_32bit, const float* w2, float eps2, float offset2, void* stream) {
     if (rows == 0) return MG_OK;
     MG_REQUIRE(rows > 0 && width > 0 && x && a && w, "norm_add: bad sizes");
     MG_REQUIRE(entry_slot == nullptr || (top > 0 && n_slots > 0 && b == nullptr && !clear && sa == 1.f),
                "norm_add: a sum over entries takes neither a second input nor a factor, and is not cleared");
+    MG_REQUIRE((w2 == nullptr || out_rows != nullptr) && (!rows_32bit || w2 != nullptr), "norm_add: rows that nothing is written to");
     const NormInput in{a, sa, b, sb, entry_slot, top, n_slots};
-    const NormOutput out{x, w, eps, offset, scale, center, clear, (bf16*)out_rows};
+    const NormOutput out{x, w, eps, offset, scale, center, clear, rows_32bit ? nullptr : (bf16*)out_rows,
+                         rows_32bit ? (float*)out_rows : nullptr, w2, eps2, offset2};
     const bool vec = width % 4 == 0 && width <= ROW_THREADS * MAX_ROW_VECS * 4 && (uintptr_t)x % 16 == 0 && (uintptr_t)a % 16 == 0 &&
-                     (uintptr_t)b % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out_rows % 4 == 0;
+                     (uintptr_t)b % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out_rows % (w2 ? 16 : 4) == 0 && (uintptr_t)w2 % 16 == 0;
     const int per_thread = ceil_div(width / 4, ROW_THREADS);
     auto vec_kernel = per_thread <= 1 ? norm_add_vec_kernel<1> : per_thread <= 2 ? norm_add_vec_kernel<2>
                     : per_thread <= 4 ? norm_add_vec_kernel<4> : norm_add_vec_kernel<8>;

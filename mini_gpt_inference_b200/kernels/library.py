@@ -23,9 +23,11 @@ _SIGNATURES = {
     "mg_guards_enabled": [],
     "mg_embed": [_P, _P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _F, _P],
     "mg_scale": [_P, ctypes.c_longlong, _F, _P],
-    "mg_head_prepare": [_P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _P, _P, _P],
+    "mg_head_prepare": [_P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _P, _P,
+                        _F, ctypes.c_double, _P],
+    "mg_latent_pair_prepare": [_P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _F, _P, _P, _P, _I, _I, _I, _P],
     "mg_paged_attention_general": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _I, _F,
-                                   _I, _I, _I, _P, _I, _F, _P, _I, _P],
+                                   _I, _I, _I, _P, _I, _F, _P, _I, _I, _P],
     "mg_streams_read": [_P, _P, _P, _P, _I, ctypes.c_longlong, _P],
     "mg_streams_write": [_P, _P, _P, _P, _P, _P, _P, _I, ctypes.c_longlong, _P],
     "mg_streams_spread": [_P, _P, _I, ctypes.c_longlong, _P],
@@ -34,14 +36,14 @@ _SIGNATURES = {
     "mg_rotate_heads": [_P, _I, _I, _I, _P, _P, _F, _I, _P],
     "mg_gated_recurrence": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, ctypes.c_longlong, _P, _I, _I, _I, _I, _I, _I, _P],
     "mg_token_shift_mix": [_P, _P, _P, _P, _P, _P, _P, _P, ctypes.c_longlong, _P, _I, _I, _I, _I, _I, _I, _P],
-    "mg_norm_add": [_P, _P, _F, _P, _F, _P, _I, _I, _P, _I, _I, _F, _F, _I, _F, _I, _P, _P],
+    "mg_norm_add": [_P, _P, _F, _P, _F, _P, _I, _I, _P, _I, _I, _F, _F, _I, _F, _I, _P, _I, _P, _F, _F, _P],
     "mg_add_rows": [_P, _P, _P, ctypes.c_longlong, _I, _P],
     "mg_scaled_sum": [_P, _P, _F, _P, _F, ctypes.c_longlong, _I, _P],
     "mg_softcap": [_P, ctypes.c_longlong, _F, _P],
     "mg_cast_rows": [_P, _P, ctypes.c_longlong, _I, _I, _P],
     "mg_token_gate": [_P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P],
     "mg_latent_prepare": [_P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P],
-    "mg_head_linear": [_P, _I, _I, _I, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "mg_head_linear": [_P, _I, _I, _I, _P, _I, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "mg_causal_conv_silu": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, ctypes.c_longlong, _P, _I, _I, _I, _I, _I, _I, _P],
     "mg_conv_state_update": [_P, _I, _I, _P, _P, _P, _P, _P, ctypes.c_longlong, _I, _I, _I, _I, _I, _P],
     "mg_gated_group_norm": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _P],
@@ -57,11 +59,11 @@ _SIGNATURES = {
     "mg_head_norm_gate": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _P],
     "mg_moe_route_scored": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     "mg_attention_mma": [_P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F,
-                         _I, _I, _I, _I, _I, _I, _P, _I, _F, _P, _I, _P],
+                         _I, _I, _I, _I, _I, _I, _P, _I, _F, _P, _I, _I, _P],
     "mg_attention_wide": [_P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I,
                           _I, _I, _F, _P, _P],
     "mg_attention_wide_tiles": [_I, _I],
-    "mg_moe_route": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "mg_moe_route": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     "mg_moe_group": [_P, _I, _I, _P, _P, _P, _P],
     "mg_moe_gemm": [_P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P],
     "mg_moe_combine": [_P, _P, _I, _P, _I, _I, _I, _P],

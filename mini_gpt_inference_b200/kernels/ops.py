@@ -886,14 +886,18 @@ class CudaOps:
         return out
 
     def head_prepare(self, proj, n_head, n_kv_head, head_dim, v_dim, q_off, k_off, v_off, unit_norm, eps,
-                     cache, slots, positions, v_other=None, blend=None, q_gain=None, k_gain=None):
+                     cache, slots, positions, v_other=None, blend=None, q_gain=None, k_gain=None, q_temperature=None):
         """Between a fused projection and the attention, in one kernel (``q_gain`` / ``k_gain``: 32-bit gains of
         ``head_dim`` numbers on the unit-RMS query and key heads): query and key heads of
         ``proj`` rows divided by their root mean square (``unit_norm``; queries in place), values
         blended with ``v_other`` (a 2-D view whose rows' first columns are the other values of the
         same tokens; ``blend`` a 32-bit scalar on the device), keys and values written to the cache
-        rows ``slots`` (``cache`` None or read-only: nothing is written)."""
+        rows ``slots`` (``cache`` None or read-only: nothing is written).  ``q_temperature`` ``(coef, every)``: the query heads
+        of position ``p`` are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``."""
         self._want(proj, None, "projection rows", 2)
+        coef, every = q_temperature if q_temperature is not None else (0.0, 0.0)
+        if q_temperature is not None and self._want(positions, torch.int32, "positions", 1).numel() != proj.shape[0]:
+            raise KernelLibraryError("head_prepare: one position per row")
         is_bf16 = self._is_bf16(proj)
         args_other = [None, 0, None]
         if v_other is not None:
@@ -915,7 +919,7 @@ class CudaOps:
             _ptr(proj), proj.shape[1], proj.shape[0], n_head, n_kv_head, head_dim, v_dim, q_off, k_off, v_off,
             1 if unit_norm else 0, float(eps), *args_other, pages[0], _ptr(positions), pages[1], pages[2],
             pages[3], pages[4], is_bf16, _ptr(self._gain(q_gain, head_dim)), _ptr(self._gain(k_gain, head_dim)),
-            self._stream()), "head_prepare")
+            float(coef), float(every), self._stream()), "head_prepare")
 
     def _gain(self, gain, size):
         if gain is not None and self._want(gain, torch.float32, "head gain", 1).numel() != size:
@@ -931,13 +935,16 @@ class CudaOps:
         is taken off the score of query ``i`` and key ``j``; ``block``: a query sees only the keys
         of its own block of that many positions; ``softcap``: a score ``s`` (scale included) becomes
         ``softcap * tanh(s / softcap)``; ``sinks`` (32-bit, one per head): ``exp(sink)`` is added to the
-        softmax's denominator.  A cache whose values live in its key rows is read that way.  Returns
+        softmax's denominator.  A cache whose values live in its key rows is read that way, and one that keeps first tokens
+        beside its window (``keep_first``) has them in every query's sight.  Returns
         ``[tokens, n_head * v_dim]``."""
         if sinks is not None and self._want(sinks, torch.float32, "sinks", 1).numel() != n_head:
             raise KernelLibraryError("attention: one sink per head")
         softcap = float(softcap or 0.0)
         in_keys = bool(getattr(cache, "values_in_keys", False))
-        plain = softcap == 0.0 and sinks is None and not in_keys      # what the tensor-core kernels take
+        keep_first = int(getattr(cache, "keep_first", 0))
+        # what the tcgen05 prompt attention takes
+        plain = softcap == 0.0 and sinks is None and not in_keys and keep_first == 0
         if slopes is not None and self._want(slopes, torch.float32, "slopes", 1).numel() != n_head:
             raise KernelLibraryError("attention: one slope per head")
         block = int(block or 0)
@@ -978,7 +985,7 @@ class CudaOps:
             group = n_head // n_kv_head
             args = None
             if single:
-                keys, splits = self._key_ranges(int(ctx.max_ctx_after), int(cache.window or 0), block)
+                keys, splits = self._key_ranges(int(ctx.max_ctx_after), int(cache.window or 0), block, keep_first)
                 floats = self.lib.mg_attention_mma_scratch_floats(n, n_head, v_dim, splits)
                 scratch = torch.empty((floats,), dtype=torch.float32, device=self.device)
                 # (measured at batch 8, context 2,048: the ranges merged by a second kernel, 0.273 ms a
@@ -995,13 +1002,13 @@ class CudaOps:
                     _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out), args[0], args[1], n, table.shape[0],
                     n_head, n_kv_head, head_dim, v_dim, cache.page_tokens, table.shape[1], int(cache.window or 0),
                     float(scale), cache.k_pages.shape[0], *args[2:], _ptr(slopes), block, softcap, _ptr(sinks),
-                    head_dim if in_keys else 0, self._stream())
+                    head_dim if in_keys else 0, keep_first, self._stream())
                 if code != library.UNSUPPORTED:
                     self._run(code, "paged_attention (tensor cores, general)")
                     if single and args[1] is None:
                         self.launches += 1                       # the merge of the ranges as a kernel of its own
                     return out
-        if q.dtype == torch.bfloat16 and self.use_tensor_cores and self.use_mma_attention and in_keys and not biased:
+        if q.dtype == torch.bfloat16 and self.use_tensor_cores and self.use_mma_attention and in_keys and not biased and keep_first == 0:
             # rows too wide for that kernel's registers (cached latents of several hundred features): tiles of 32
             # (token, head) rows whose queries wait in shared memory
             single = bool(getattr(ctx, "decode_only", False))
@@ -1032,17 +1039,18 @@ class CudaOps:
             _ptr(ctx.positions), _ptr(out), n, n_head, n_kv_head, head_dim, v_dim, _ptr(gate),
             gate.stride(0) if gate is not None else 0, cache.page_tokens, table.shape[1], int(cache.window or 0),
             float(scale), cache.k_pages.shape[0], table.shape[0], self._is_bf16(q), _ptr(slopes), block,
-            softcap, _ptr(sinks), head_dim if in_keys else 0, self._stream()), "paged_attention (general)")
+            softcap, _ptr(sinks), head_dim if in_keys else 0, keep_first, self._stream()), "paged_attention (general)")
         return out
 
-    def _key_ranges(self, max_context, window, block):
+    def _key_ranges(self, max_context, window, block, keep_first=0):
         """Keys per range and ranges per token for single tokens with contexts of up to ``max_context`` keys.  With a
         window or a block mask a token's keys begin at its own first position: ranges are counted from the key block of
-        64 that holds it, so they cover at most the window's (the block's) length and 63 keys in front of it."""
+        64 that holds it, so they cover at most the window's (the block's) length and 63 keys in front of it, behind the blocks that hold first tokens
+        which stay in sight."""
         span = max_context
         for reach in (window, block):
             if reach > 0:
-                span = min(span, reach + 64)
+                span = min(span, reach + 64 + -(-keep_first // 64) * 64)
         keys = self.lib.mg_attention_mma_split_keys(span)
         return keys, max(1, -(-span // keys))
 
@@ -1196,11 +1204,12 @@ class CudaOps:
         return out
 
     def norm_add(self, residual32, y32, weight, eps, offset=0.0, center=False, norm_scale=1.0, other32=None, scale=1.0,
-                 other_scale=1.0, clear=False, rows_dtype=None):
+                 other_scale=1.0, clear=False, rows_dtype=None, then=None):
         """``residual32 += norm_scale * norm(scale * y32 [+ other_scale * other32]) * (offset + weight)``, in place, 32-bit:
         an RMS norm, or with ``center`` a layer norm without a shift.  ``y32`` may be an ``EntrySum``: the norm then takes
         the sum on its way.  ``clear``: ``y32`` (and ``other32``) are left as zeros, ready for the next sublayer to add
-        into.  With ``rows_dtype`` the new stream is also returned in that type (``residual32`` itself if 32-bit)."""
+        into.  With ``rows_dtype`` the new stream is also returned in that type (``residual32`` itself if 32-bit); with ``then``
+        ``(weight, eps, offset)`` an RMS norm of it is, ``x / sqrt(mean(x^2) + eps) * (offset + weight)``."""
         self._want(residual32, torch.float32, "residual", 2)
         entries = [None, 0, 0]
         terms = y32
@@ -1218,14 +1227,18 @@ class CudaOps:
                 or (other32 is not None and other32.shape != y32.shape)):
             raise KernelLibraryError("norm_add: shapes do not fit")
         rows = residual32 if rows_dtype == torch.float32 else None
-        if rows_dtype == torch.bfloat16:
-            rows = torch.empty(residual32.shape, dtype=rows_dtype, device=self.device)
-        elif rows_dtype not in (None, torch.float32):
+        if rows_dtype not in (None, torch.float32, torch.bfloat16) or (then is not None and rows_dtype is None):
             raise KernelLibraryError(f"norm_add: rows in {rows_dtype}")
+        w2, eps2, offset2 = then if then is not None else (None, 0.0, 0.0)
+        if w2 is not None and self._want(w2, torch.float32, "norm weight", 1).numel() != residual32.shape[1]:
+            raise KernelLibraryError("norm_add: the weight of the norm behind does not match the width")
+        if rows_dtype == torch.bfloat16 or then is not None:
+            rows = torch.empty(residual32.shape, dtype=rows_dtype, device=self.device)
         self._run(self.lib.mg_norm_add(
             _ptr(residual32), _ptr(terms), float(scale), _ptr(other32), float(other_scale), *entries, _ptr(weight),
             residual32.shape[0], residual32.shape[1], float(eps), float(offset), 1 if center else 0, float(norm_scale),
-            1 if clear else 0, _ptr(rows) if rows_dtype == torch.bfloat16 else None, self._stream()), "norm_add")
+            1 if clear else 0, None if rows is residual32 else _ptr(rows), 1 if then is not None and rows_dtype == torch.float32 else 0,
+            _ptr(w2), float(eps2), float(offset2), self._stream()), "norm_add")
         return rows
 
     def rmsnorm_add(self, residual32, y32, weight, eps, offset=0.0, other32=None, scale=1.0, other_scale=1.0, clear=False):
@@ -1343,23 +1356,46 @@ class CudaOps:
             self._is_bf16(proj), 1 if neighbours else 0, float(magnitude), self._stream()), "latent_prepare")
         return q
 
+    def latent_pair_prepare(self, proj, q_off, q_rank, q_gain, low_off, rank, gain, eps, cache, slots, positions):
+        """For an attention over cached latents whose queries come from a latent of their own: the ``rank`` numbers of
+        ``proj`` from ``low_off``, RMS-normed with ``gain``, go to the token's cache row; the ``q_rank`` numbers from
+        ``q_off``, normed with ``q_gain``, are returned as ``[tokens, q_rank]``."""
+        self._want(proj, None, "projection rows", 2)
+        self._want(positions, torch.int32, "positions", 1)
+        self._want(slots, torch.int32, "slot_mapping", 1)
+        self._want(cache.k_pages, proj.dtype, "k_pages", 4)
+        for g, size in ((q_gain, q_rank), (gain, rank)):
+            if self._want(g, torch.float32, "latent gain", 1).numel() != size:
+                raise KernelLibraryError("latent_pair_prepare: a gain does not match its latent")
+        if (not cache.writes or not getattr(cache, "values_in_keys", False)
+                or tuple(cache.k_pages.shape[1:]) != (1, cache.page_tokens, rank)):
+            raise KernelLibraryError("latent_pair_prepare: page storage does not match the latent")
+        out = torch.empty((proj.shape[0], q_rank), dtype=proj.dtype, device=self.device)
+        self._run(self.lib.mg_latent_pair_prepare(
+            _ptr(proj), proj.shape[1], proj.shape[0], q_off, q_rank, _ptr(q_gain), _ptr(out), low_off, rank, _ptr(gain),
+            float(eps), _ptr(positions), _ptr(slots), _ptr(cache.k_pages), cache.page_tokens, cache.k_pages.shape[0],
+            self._is_bf16(proj), self._stream()), "latent_pair_prepare")
+        return out
+
     def head_linear(self, x, x_off, x_head, weight, rows_are_inputs, n_head, n_in, n_out, gate=None, out=None, out_off=0,
                     out_head=None):
         """One small matrix per head: ``out[n, h, j] = sum_i x[n, h, i] * W_h[j, i]`` with ``weight``
         ``[n_head * n_out, n_in]``, or, with ``rows_are_inputs``, ``sum_i x[n, h, i] * W_h[i, j]`` with ``weight``
         ``[n_head * n_in, n_out]``.  Head h's inputs are the columns ``x_off + h * x_head ..`` of ``x``; its outputs go
         to the columns ``out_off + h * out_head ..`` of ``out`` (a new ``[tokens, n_head * n_out]`` tensor unless
-        given).  ``gate`` (a 2-D view, ``n_head * n_out`` columns): the outputs times its logistic function."""
+        given).  ``gate`` (a 2-D view of ``n_head * n_out`` columns, or of ``n_head``, one for all of a head's outputs): the
+        outputs times its logistic function."""
         self._want(x, weight.dtype, "head inputs", 2)
         self._want(weight, None, "head matrices", 2)
         if weight.shape != ((n_head * n_in, n_out) if rows_are_inputs else (n_head * n_out, n_in)):
             raise KernelLibraryError("head_linear: the matrices do not fit the heads")
         n = x.shape[0]
         if gate is not None and (gate.dtype != x.dtype or gate.dim() != 2 or gate.stride(1) != 1
-                                 or gate.shape != (n, n_head * n_out)):
+                                 or gate.shape not in ((n, n_head * n_out), (n, n_head))):
             raise KernelLibraryError("head_linear: the gate does not fit the heads")
         if out is None:
-            out, out_off, out_head = torch.empty((n, n_head * n_out), dtype=x.dtype, device=self.device), 0, n_out
+            out_head = n_out if out_head is None else out_head
+            out = torch.empty((n, out_off + n_head * out_head), dtype=x.dtype, device=self.device)
         else:
             self._want(out, x.dtype, "head outputs", 2)
             out_head = n_out if out_head is None else out_head
@@ -1367,7 +1403,8 @@ class CudaOps:
                 raise KernelLibraryError("head_linear: one output row per token")
         self._run(self.lib.mg_head_linear(
             _ptr(x), x.shape[1], x_off, x_head, _ptr(weight), 1 if rows_are_inputs else 0, _ptr(gate),
-            gate.stride(0) if gate is not None else 0, _ptr(out), out.shape[1], out_off, out_head, n, n_head, n_in, n_out,
+            gate.stride(0) if gate is not None else 0, 1 if gate is not None and gate.shape[1] == n_head else 0, _ptr(out),
+            out.shape[1], out_off, out_head, n, n_head, n_in, n_out,
             self._is_bf16(x), self._stream()), "head_linear")
         return out
 
@@ -1414,12 +1451,16 @@ class CudaOps:
         return out
 
     # ---- routed experts ---------------------------------------------------------------------------
-    def moe_route(self, y, router_weight, gate_weight, positions, top, always=0):
+    def moe_route(self, y, router_weight, gate_weight, positions, top, always=0, scoring="softmax_top", scale=1.0):
         """Router of a feed-forward of experts: returns (ids [tokens, top] int32, weights [tokens,
         top] 32-bit, gate [tokens] 32-bit or None): the ``top`` largest of ``router_weight @ y``
         with the softmax over them, and the logistic function of ``gate_weight . y``.  ``always`` experts behind the
         router's own (numbers ``experts ..``) join every token's chosen ones as further columns of ids and weights, with
-        the gate's value (1 without one) as their weight; then no gate is returned."""
+        the gate's value (1 without one) as their weight; then no gate is returned.  ``scoring`` ``"sigmoid"``: the experts
+        with the largest ``sigmoid(z)``, their weights ``scale`` times that, not renormalised (else ``scale`` times the
+        softmax)."""
+        if scoring not in ("sigmoid", "softmax_top"):
+            raise KernelLibraryError(f"moe_route: scoring {scoring!r}")
         self._want(y, None, "router input", 2)
         self._want(router_weight, torch.float32, "router weight", 2)
         n, width = y.shape
@@ -1436,7 +1477,8 @@ class CudaOps:
             if not always:
                 gate = torch.empty((n,), dtype=torch.float32, device=self.device)
         self._run(self.lib.mg_moe_route(_ptr(y), _ptr(router_weight), _ptr(gate_weight), _ptr(positions), _ptr(ids),
-                                        _ptr(weights), _ptr(gate), n, width, experts, top, int(always), self._is_bf16(y),
+                                        _ptr(weights), _ptr(gate), n, width, experts, top, int(always),
+                                        1 if scoring == "sigmoid" else 0, float(scale), self._is_bf16(y),
                                         self._stream()), "moe route")
         return ids, weights, gate
 
@@ -1471,11 +1513,12 @@ class CudaOps:
                                                self._is_bf16(y), self._stream()), "moe route (scored)")
         return ids, weights, gate
 
-    def moe_experts(self, y, ids, weights, w_in, w_out, activation="silu", limit=0.0, gated=True):
+    def moe_experts(self, y, ids, weights, w_in, w_out, activation="silu", limit=0.0, gated=True, weigh_input=False):
         """``sum_k weights[t, k] * expert(ids[t, k])(y[t])`` as an ``EntrySum`` (every entry's product apart), with expert
         e as ``w_out[e] @ (silu(w_in[e][:F] @ y) * (w_in[e][F:] @ y))``, ``w_in`` [E, 2F, C], ``w_out`` [E, C, F], or, not
         ``gated``, ``w_out[e] @ act(w_in[e] @ y)`` with ``w_in`` [E, F, C] (``activation``: ``relu_sq``, ``gelu_tanh``,
-        ``silu``).  Tokens are grouped by expert on the device; the host never learns the counts."""
+        ``silu``).  With ``weigh_input`` a weight multiplies what its expert reads: ``expert(weights[t, k] * y[t])``.  Tokens are
+        grouped by expert on the device; the host never learns the counts."""
         self._want(y, w_in.dtype, "expert input", 2)
         self._want(w_in, None, "expert matrices (in)", 3)
         self._want(w_out, w_in.dtype, "expert matrices (out)", 3)
@@ -1493,22 +1536,23 @@ class CudaOps:
         self._run(self.lib.mg_moe_group(_ptr(ids), entries, experts, _ptr(offsets), _ptr(slot_entry), _ptr(entry_slot),
                                         self._stream()), "moe group")
         hidden = torch.empty((entries, inner), dtype=y.dtype, device=self.device)
-        self._run(self.lib.mg_moe_gemm(_ptr(y), width, _ptr(w_in), _ptr(offsets), _ptr(slot_entry), top, None,
-                                       _ptr(hidden), experts, n, inner, width, n, 1 if gated else 2, is_bf16, act, float(limit),
+        self._run(self.lib.mg_moe_gemm(_ptr(y), width, _ptr(w_in), _ptr(offsets), _ptr(slot_entry), top,
+                                       _ptr(weights) if weigh_input else None, _ptr(hidden), experts, n, inner, width, n, 1 if gated else 2, is_bf16, act, float(limit),
                                        self._stream()),
                   "moe experts (in)")
         out = torch.empty((entries, width), dtype=torch.float32, device=self.device)
         self._run(self.lib.mg_moe_gemm(_ptr(hidden), inner, _ptr(w_out), _ptr(offsets), _ptr(slot_entry), top,
-                                       _ptr(weights), _ptr(out), experts, n, width, inner, entries, 0, is_bf16, 0, 0.0,
+                                       None if weigh_input else _ptr(weights), _ptr(out), experts, n, width, inner, entries, 0, is_bf16, 0, 0.0,
                                        self._stream()), "moe experts (out)")
         return EntrySum(out, entry_slot)
 
-    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0, gated=True):
+    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0, gated=True,
+                             weigh_input=False):
         """``residual32[t] += `` the sum that ``moe_experts`` describes."""
         self._want(residual32, torch.float32, "residual", 2)
         if tuple(residual32.shape) != tuple(y.shape):
             raise KernelLibraryError("moe_experts: the residual does not fit")
-        y = self.moe_experts(y, ids, weights, w_in, w_out, activation, limit, gated)
+        y = self.moe_experts(y, ids, weights, w_in, w_out, activation, limit, gated, weigh_input)
         n, width = y.shape
         self._run(self.lib.mg_moe_combine(_ptr(y.terms), _ptr(y.entry_slot), y.entry_slot.shape[1], _ptr(residual32), n, width,
                                           y.terms.shape[0], self._stream()), "moe combine")

@@ -9,7 +9,8 @@ between a norm and the following projection is the compute dtype.
 Interfaces (what a new part must provide):
 
 * Norm:             ``forward(ctx, x32) -> y``            y in ctx.act_dtype, same shape; a norm that can stand behind
-                    a sublayer also has ``add_normed`` (reads the sublayer's output, adds into the stream)
+                    a sublayer also has ``add_normed`` (reads the sublayer's output, adds into the stream; it may
+                    hand on the rows that the norm in front of the next sublayer makes of the new stream)
 * PositionEncoding: ``table()`` (rows added to the token embedding, or None),
                     ``rotate(ctx, qkv, n_head, n_kv_head, head_dim)`` (in place on the q and
                     k columns of the fused projection; default no-op),
@@ -73,16 +74,20 @@ class Part:
             setattr(self, local, tensors.get(full_name))
 
     @staticmethod
-    def add_output(ctx, rows, weight, residual32):
-        """A part's last projection: ``rows W^T`` added into ``residual32`` in place, or, without one, returned in
+    def add_output(ctx, rows, weight, residual32, bias=None):
+        """A part's last projection: ``rows W^T + bias`` added into ``residual32`` in place, or, without one, returned in
         32-bit."""
         if residual32 is None:
-            return ctx.ops.linear(rows, weight, None, "none", torch.float32)
-        ctx.ops.linear_residual(rows, weight, None, residual32)
+            return ctx.ops.linear(rows, weight, bias, "none", torch.float32)
+        ctx.ops.linear_residual(rows, weight, bias, residual32)
         return None
 
 
 class Norm(Part):
+    # True for a norm whose kernel behind a sublayer can also apply a second such norm to the new stream
+    # (``add_normed(..., then=the other norm)``).
+    chains = False
+
     def forward(self, ctx, x32):
         raise NotImplementedError
 

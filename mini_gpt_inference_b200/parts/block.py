@@ -11,8 +11,9 @@ returns the tensor that holds it at the end (or nothing, if that is the one it w
 ``pre_norm_mixer_only``: ``x += mixer(norm1(x))``, for a layer without a feed-forward.
 ``sandwich_norm``: a norm on both sides of each sublayer, ``x += norm1b(mixer(norm1(x)))``, then, if the layer has a
 feed-forward, ``x += norm2b(ff(norm2(x)))``, then, if it has one, the layer's token input (``side_input``), which
-reads the stream and the step's tokens and adds into the stream.  The sublayers add their output into a zeroed
-32-bit buffer; the norm behind them reads it and adds into the stream in one kernel.
+reads the stream and the step's tokens and adds into the stream.  The norm behind a sublayer reads its output (what the
+sublayer returns, or, of one that can only add, a zeroed 32-bit buffer that it added into) and adds into the stream in
+one kernel; where the feed-forward takes plain rows, that kernel also applies the norm in front of it.
 ``post_norm``: norms behind the sublayers only, ``x += r * norm1(mixer(x))``, then, if the layer has a feed-forward,
 ``x += r * norm2(ff(x))``, with ``r`` the layer's setting ``residual_scale``.  The sublayers read the stream itself, in the
 compute dtype; the norm behind a sublayer writes that copy of the new stream on its way, for the next sublayer or layer.
@@ -97,14 +98,24 @@ register_arrangement("pre_norm_mixer_only")(pre_norm_mixer_only)
 def sandwich_norm(ctx, layer: Layer, cache, residual32):
     x = residual32
     rows, width = x.shape
-    # one zeroed buffer serves every sublayer of the pass: the norm behind a sublayer leaves it as zeros again
-    zeros = ctx.ops.zeros32(rows, width, ctx)
-    y = stream_after(layer.mixer.forward(ctx, cache, _normed(ctx, layer.norm1, layer.mixer, x), zeros), zeros)
-    layer.norm1b.add_normed(ctx, y, x, clear=y is zeros)
-    ff = layer.get("feed_forward")
+
+    def add(part, norm, run, then=None):
+        chained = {} if then is None else {"then": then}
+        if part.returns_output:
+            return norm.add_normed(ctx, run(None), x, **chained)
+        # one zeroed buffer serves every sublayer of the pass: the norm behind a sublayer leaves it as zeros again
+        zeros = ctx.ops.zeros32(rows, width, ctx)
+        y = stream_after(run(zeros), zeros)
+        return norm.add_normed(ctx, y, x, clear=y is zeros, **chained)
+    mixer, ff = layer.mixer, layer.get("feed_forward")
+    then = None
+    if ff is not None and not ff.accepts_deferred_norm and layer.norm1b.chains and layer.norm2.chains:
+        then = layer.norm2
+    u = add(mixer, layer.norm1b, lambda into: mixer.forward(ctx, cache, _normed(ctx, layer.norm1, mixer, x), into), then)
     if ff is not None:
-        y = stream_after(ff.forward(ctx, _normed(ctx, layer.norm2, ff, x), zeros), zeros)
-        layer.norm2b.add_normed(ctx, y, x, clear=y is zeros)
+        if then is None:
+            u = _normed(ctx, layer.norm2, ff, x)
+        add(ff, layer.norm2b, lambda into: ff.forward(ctx, u, into))
     side = layer.get("side_input")
     if side is not None:
         side.forward(ctx, x)

@@ -37,7 +37,11 @@ scaled nor capped); ``value_unit_norm`` (every value head is divided by its root
 without a gain, and cached so); ``value_rot`` (the value of position ``j``, after that norm, turns by ``j`` over all
 its features, feature ``m`` paired with ``m + v_head_dim / 2``, angle ``j * rot_base ** (-2 m / v_head_dim)``, and is
 cached so; every head's output at position ``i`` is turned back by ``-i`` before the gate and the output projection,
-so that a value enters the sum turned by its distance to the query).
+so that a value enters the sum turned by its distance to the query); ``keep_first`` (with a ``window``: the first
+``keep_first`` tokens of the sequence stay in every query's sight, with their true positions; the cache keeps their pages);
+``unit_sink`` (one more term of 1 in the softmax's denominator, a sink whose score is 0 for every head);
+``query_temperature=(coef, every)`` (the query of position ``p`` is multiplied by
+``1 + coef * ln(floor((p + 1) / every) + 1)``, after the norm if there is one).
 
 Positions do not enter otherwise unless the model's position encoding rotates q and k.  The four
 matrices are stored apart in the checkpoint (``q``, ``k``, ``v``, ``g``, then ``o`` and the
@@ -62,6 +66,7 @@ VALUE_SOURCE = "attention_value_source"     # key in ctx.shared
 class GatedUnitAttention(Mixer):
     graph_safe = True      # launches kernels only; nothing is decided on the host per step
     accepts_deferred_norm = True
+    returns_output = True
 
     def __init__(self, prefix: str, width: int, n_head: int, head_dim: int, n_kv_head: int | None = None,
                  v_head_dim: int | None = None, scale: float | None = None, eps: float = 1e-6,
@@ -72,7 +77,8 @@ class GatedUnitAttention(Mixer):
                  values: str = "projected", slope_rate: float | None = None, block_mask: int | None = None,
                  init: str = "normal", norm_scope: str = "head", rot_dims: int = 0, rot_base: float = 10000.0,
                  softcap: float | None = None, sink: bool = False, value_unit_norm: bool = False,
-                 value_rot: bool = False) -> None:
+                 value_rot: bool = False, keep_first: int = 0, unit_sink: bool = False,
+                 query_temperature: tuple | None = None) -> None:
         super().__init__(prefix)
         self.width, self.n_head, self.head_dim = width, n_head, head_dim
         self.n_kv_head = n_head if n_kv_head is None else n_kv_head
@@ -116,7 +122,18 @@ class GatedUnitAttention(Mixer):
         if self.turns and unit_norm and norm_scope == "head":
             raise ValueError("rotary positions go with the projection-wide norm or with none")
         self.softcap = None if softcap is None else float(softcap)
-        self.has_sink = bool(sink)
+        if sink and unit_sink:
+            raise ValueError("a learned sink and a sink of 1: one of them")
+        self.has_sink, self.unit_sink = bool(sink), bool(unit_sink)
+        if keep_first < 0 or (keep_first and window is None):
+            raise ValueError("keep_first goes with a window")
+        self.keep_first = int(keep_first)
+        self.query_temperature = None
+        if query_temperature is not None:
+            coef, every = query_temperature
+            if self.turns or every <= 0:
+                raise ValueError("query_temperature goes with heads that do not turn and with a positive step")
+            self.query_temperature = (float(coef), float(every))
         self.has_bias, self.has_norm_weights, self.values_are_keys = bool(self.biased), bool(norm_weights), values == "keys"
         self.slope_rate = None if slope_rate is None else float(slope_rate)
         self.block_mask = block_mask
@@ -199,21 +216,24 @@ class GatedUnitAttention(Mixer):
             self.slopes = torch.tensor(slopes, dtype=torch.float64).to(dtype=torch.float32, device=self.out_weight.device)
         blend = tensors.get(self._name("blend")) if self.value_blend == "blend" else None
         self.blend = blend.reshape(1).contiguous() if blend is not None else None
+        if self.unit_sink and self.out_weight is not None:
+            self.sinks = torch.zeros(self.n_head, dtype=torch.float32, device=self.out_weight.device)     # exp(0) = 1
 
     def cache_spec(self):
         return PagedKVSpec(self.n_kv_head, self.head_dim, self.window, self.cache_page_tokens,
                            self.cache_pages,
-                           None if self.v_head_dim == self.head_dim else self.v_head_dim, self.block_mask)
+                           None if self.v_head_dim == self.head_dim else self.v_head_dim, self.block_mask,
+                           self.keep_first)
 
     def plan_step(self, batch, plan, ops) -> None:
         # where keys and values have one size, the kernel set may cut prompt portions into the tiles of
         # its tiled attention kernel (the same work list as the plain causal attention's)
         planner = getattr(ops, "plan_prompt_attention", None)
         if (planner is not None and self.head_dim == self.v_head_dim and self.slopes is None and self.block_mask is None
-                and self.softcap is None and not self.has_sink):
+                and self.softcap is None and not self.has_sink and not self.unit_sink and not self.keep_first):
             planner(batch, plan, self.n_head, self.n_kv_head, self.head_dim)
 
-    def forward(self, ctx, cache, y, residual32) -> None:
+    def forward(self, ctx, cache, y, residual32):
         ops = ctx.ops
         proj = ops.linear(y, self.fused_weight, self.fused_bias, "none", ctx.act_dtype)
         if self.position is not None:
@@ -236,6 +256,8 @@ class GatedUnitAttention(Mixer):
                                self.v_off, self.unit_norm, self.eps, self.rot_dims, self.freq, cache,
                                ctx.slot_mapping[cache.group], ctx.positions, **extra)
         else:
+            if self.query_temperature is not None:
+                extra["q_temperature"] = self.query_temperature
             ops.head_prepare(proj, self.n_head, self.n_kv_head, self.head_dim, self.v_head_dim, 0, self.k_off,
                              self.v_off, self.unit_norm, self.eps, cache, ctx.slot_mapping[cache.group],
                              ctx.positions, v_other=other, blend=blend, **extra)
@@ -253,4 +275,4 @@ class GatedUnitAttention(Mixer):
                                           self.scale, cache, ctx, gate=gate, **extra)
         if self.value_rot:
             ops.rotate_heads(out, self.n_head, self.v_head_dim, self.v_freq, ctx.positions, -1.0)
-        ops.linear_residual(out, self.out_weight, self.out_bias, residual32)
+        return self.add_output(ctx, out, self.out_weight, residual32, self.out_bias)

@@ -8,7 +8,10 @@ position (rotary; feature ``i`` pairs with ``i + rot_dim / 2``, angle ``position
 ``[W_uk,a c | shared part]``, its value ``W_uv,a c``, its score ``scale * (q_plain . k_plain + q_rot . k_rot)``;
 softmax over positions up to the query's own (``window``: the last ``window`` of them, its own included; ``sink``: a
 learned number per head whose exponential joins the denominator); the concatenated heads times ``sigmoid(W_g h)`` if
-``gate``, then ``W_o``.
+``gate`` (``"head"``: ``W_g h`` has one number per head, which all of the head's features share), then ``W_o``.
+
+With ``q_rank`` the queries come from a latent of their own: ``c_q = W_dq h`` (``q_rank`` numbers, RMS-normed with a gain),
+``q = W_uq c_q``; such heads do not turn (``rot_dim`` 0).  One kernel norms both latents of a token.
 
 Only ``[c | shared part]`` is cached, one row per token whatever the number of heads.  Scores are taken
 against those rows themselves: a query's plain part is first carried into the latent's space with its head's
@@ -28,7 +31,7 @@ from .base import Mixer, register_mixer
 from .rotary import SCALING_KEYS, rotary_frequencies
 from .spec import TensorSpec
 
-_DEFAULT_NAMES = {"q": "q", "down": "dkv", "norm": "dkv.norm", "up_k": "uk", "up_v": "uv", "gate": "g", "sink": "sink", "out": "o"}
+_DEFAULT_NAMES = {"q": "q", "q_down": "dq", "q_norm": "dq.norm", "q_up": "uq", "down": "dkv", "norm": "dkv.norm", "up_k": "uk", "up_v": "uv", "gate": "g", "sink": "sink", "out": "o"}
 
 
 @register_mixer("latent_attention")
@@ -38,10 +41,10 @@ class LatentAttention(Mixer):
     returns_output = True
 
     def __init__(self, prefix: str, width: int, n_head: int, head_dim: int, rot_dim: int, v_head_dim: int, kv_rank: int,
-                 scale: float, eps: float, rot_base: float = 10000.0, gate: bool = True, own_latents: bool = True,
+                 scale: float, eps: float, rot_base: float = 10000.0, gate: bool | str = True, own_latents: bool = True,
                  cache_page_tokens: int | None = None, cache_pages: int | None = None, names: dict | None = None,
                  init: str = "normal", rot_pairs: str = "halves", rot_scaling: dict | None = None,
-                 window: int | None = None, sink: bool = False, position=None) -> None:
+                 window: int | None = None, sink: bool = False, q_rank: int | None = None, position=None) -> None:
         super().__init__(prefix)
         if rot_pairs not in ("halves", "neighbours"):
             raise ValueError(f"rot_pairs {rot_pairs!r}: halves or neighbours")
@@ -51,10 +54,15 @@ class LatentAttention(Mixer):
             raise ValueError("a layer that reads another layer's rows has that layer's window")
         if rot_dim < 0 or rot_dim % 2:
             raise ValueError(f"rot_dim {rot_dim}: an even number of features")
+        if q_rank is not None and (rot_dim or not own_latents):
+            raise ValueError("queries from a latent: heads that do not turn, in a layer that caches latents of its own")
+        if gate not in (True, False, "head"):
+            raise ValueError(f"gate {gate!r}: True, False or 'head'")
         self.width, self.n_head, self.head_dim, self.rot_dim = width, n_head, head_dim, rot_dim
         self.v_head_dim, self.kv_rank = v_head_dim, kv_rank
         self.scale, self.eps, self.rot_base = float(scale), float(eps), float(rot_base)
-        self.has_gate, self.own_latents = bool(gate), bool(own_latents)
+        self.has_gate, self.own_latents, self.head_gate = bool(gate), bool(own_latents), gate == "head"
+        self.q_rank = q_rank
         self.cache_page_tokens, self.cache_pages = cache_page_tokens, cache_pages
         self.names = {**_DEFAULT_NAMES, **(names or {})}
         self._init = init
@@ -63,8 +71,11 @@ class LatentAttention(Mixer):
         self.q_width = n_head * (head_dim + rot_dim)
         self.low_width = kv_rank + rot_dim if self.own_latents else 0
         self.o_width = n_head * v_head_dim
-        self.low_off, self.g_off = self.q_width, self.q_width + self.low_width
+        first = self.q_width if q_rank is None else q_rank
+        self.low_off, self.g_off = first, first + self.low_width
+        self.g_width = n_head if self.head_gate else self.o_width
         self.row_dim = kv_rank + rot_dim                 # a cache row, and a query head as the attention sees it
+        self.q_up = self.q_gain = None
         self.fused_weight = self.out_weight = self.up_k = self.up_v = self.latent_gain = self.freq = self.sinks = None
         self.rot_magnitude = 1.0
 
@@ -74,28 +85,37 @@ class LatentAttention(Mixer):
     def tensor_specs(self):
         init, init_out = self._init, ("residual_proj" if self._init == "normal" else self._init + "_residual")
         specs = {
-            self._name("q"): TensorSpec((self.q_width, self.width), "matrix", init),
             self._name("up_k"): TensorSpec((self.n_head * self.head_dim, self.kv_rank), "matrix", "fan_in"),
             self._name("up_v"): TensorSpec((self.o_width, self.kv_rank), "matrix", "fan_in"),
             self._name("out"): TensorSpec((self.width, self.o_width), "matrix", init_out),
         }
+        if self.q_rank is None:
+            specs[self._name("q")] = TensorSpec((self.q_width, self.width), "matrix", init)
+        else:
+            specs[self._name("q_down")] = TensorSpec((self.q_rank, self.width), "matrix", init)
+            specs[self._name("q_norm")] = TensorSpec((self.q_rank,), "vector", "norm_gain")
+            specs[self._name("q_up")] = TensorSpec((self.q_width, self.q_rank), "matrix", "fan_in")
         if self.own_latents:
             specs[self._name("down")] = TensorSpec((self.low_width, self.width), "matrix", init)
             specs[self._name("norm")] = TensorSpec((self.kv_rank,), "vector", "norm_gain")
         if self.has_gate:
-            specs[self._name("gate")] = TensorSpec((self.o_width, self.width), "matrix", init)
+            specs[self._name("gate")] = TensorSpec((self.g_width, self.width), "matrix", init)
         if self.has_sink:
             specs[self._name("sink")] = TensorSpec((self.n_head,), "vector", "unit_normal")
         return specs
 
     def bind(self, tensors) -> None:
-        rows = [tensors.get(self._name("q"))]
+        rows = [tensors.get(self._name("q" if self.q_rank is None else "q_down"))]
         if self.own_latents:
             rows.append(tensors.get(self._name("down")))
         if self.has_gate:
             rows.append(tensors.get(self._name("gate")))
         # one matrix for the step's one projection [q | low | g]: a layout made once, when the weights arrive
         self.fused_weight = torch.cat(rows, dim=0).contiguous() if all(r is not None for r in rows) else None
+        if self.q_rank is not None and self.fused_weight is not None:
+            # one gate number per head: rows of zeros fill the projection up to whole 16-byte groups of outputs
+            self.fused_weight = torch.nn.functional.pad(self.fused_weight, (0, 0, 0, -self.fused_weight.shape[0] % 8))
+            self.q_gain, self.q_up = tensors.get(self._name("q_norm")), tensors.get(self._name("q_up"))
         self.out_weight = tensors.get(self._name("out"))
         self.up_k, self.up_v = tensors.get(self._name("up_k")), tensors.get(self._name("up_v"))
         self.latent_gain = tensors.get(self._name("norm")) if self.own_latents else None
@@ -118,15 +138,21 @@ class LatentAttention(Mixer):
             raise RuntimeError(f"{self.prefix}: no cache entry holds the latents this layer reads")
         proj = ops.linear(y, self.fused_weight, None, "none", ctx.act_dtype)
         # queries as the attention sees them: per head [W_uk^T q_plain | turned q_rot]
-        q = ops.latent_prepare(proj, self.n_head, 0, self.head_dim, self.rot_dim, self.low_off, self.kv_rank,
-                               self.latent_gain, self.eps, self.freq, cache if self.own_latents else None,
-                               ctx.slot_mapping[cache.group], ctx.positions, neighbours=self.rot_neighbours,
-                               magnitude=self.rot_magnitude)
-        ops.head_linear(proj, 0, self.head_dim + self.rot_dim, self.up_k, True, self.n_head, self.head_dim, self.kv_rank,
-                        out=q, out_off=0, out_head=self.row_dim)
+        plain = proj
+        if self.q_rank is None:
+            q = ops.latent_prepare(proj, self.n_head, 0, self.head_dim, self.rot_dim, self.low_off, self.kv_rank,
+                                   self.latent_gain, self.eps, self.freq, cache if self.own_latents else None,
+                                   ctx.slot_mapping[cache.group], ctx.positions, neighbours=self.rot_neighbours,
+                                   magnitude=self.rot_magnitude)
+        else:
+            latent = ops.latent_pair_prepare(proj, 0, self.q_rank, self.q_gain, self.low_off, self.kv_rank,
+                                             self.latent_gain, self.eps, cache, ctx.slot_mapping[cache.group], ctx.positions)
+            plain, q = ops.linear(latent, self.q_up, None, "none", ctx.act_dtype), None
+        q = ops.head_linear(plain, 0, self.head_dim + self.rot_dim, self.up_k, True, self.n_head, self.head_dim, self.kv_rank,
+                            out=q, out_off=0, out_head=self.row_dim)
         mixed = ops.paged_attention_general(q, self.n_head, 1, self.row_dim, self.kv_rank, self.scale, cache, ctx,
                                             sinks=self.sinks)
-        gate = proj[:, self.g_off: self.g_off + self.o_width] if self.has_gate else None
+        gate = proj[:, self.g_off: self.g_off + self.g_width] if self.has_gate else None
         heads = ops.head_linear(mixed, 0, self.kv_rank, self.up_v, False, self.n_head, self.kv_rank, self.v_head_dim,
                                 gate=gate)
         return self.add_output(ctx, heads, self.out_weight, residual32)

@@ -15,11 +15,16 @@ the experts of the best ``keep`` groups be chosen.  ``activation="clamped_swish"
 ``W_down (g * sigmoid(1.702 g) * (u + 1))`` with ``g = min(W_gate y, limit)``,
 ``u = clamp(W_up y, -limit, limit)``; the shared expert has a limit of its own.
 
+``weigh="input"`` puts a chosen expert's weight on what it reads instead of what it gives, ``expert_k(weight_k y)``.  (The
+first product is linear, so the kernel multiplies its 32-bit sums, in front of the activation.)
+
 ``gated=False`` makes an expert a plain unit, ``W_down act(W_up y)`` (``activation``: ``relu_sq``, ``gelu_tanh`` or
-``silu``; no ``gate`` tensors), and the shared expert of the same form.  Its hidden features are then cut into parts as
-large as an expert's (the last one filled up with zero rows): since ``W_down act(W_up y)`` is a sum over hidden features,
-the parts are experts that every token uses with the shared gate as their weight, and the whole feed-forward is one
-grouping and two grouped products.
+``silu``; no ``gate`` tensors), and the shared expert of the same form.
+
+A shared expert without a gate matrix, or one without a gate number per token, is cut into parts of its hidden features
+as large as an expert's (the last one filled up with zero rows): since its output is a sum over hidden features, the
+parts are experts that every token uses with the shared gate (or 1) as their weight, and the whole feed-forward is one
+grouping and two grouped products, whose sum over a token's experts the norm behind the part can take on its way.
 
 In the checkpoint expert ``e`` has ``e<e>.gate``, ``e<e>.up``, ``e<e>.down`` under the part's
 prefix, the router ``router``, the shared expert ``shared.gate``, ``shared.up``, ``shared.down``
@@ -46,7 +51,7 @@ class RoutedExperts(FeedForward):
                  shared_inner: int | None = None, shared_gate: bool = True, scoring: str = "softmax_top",
                  route_scale: float = 1.0, correction: bool = False, groups: tuple | None = None,
                  activation: str = "silu", limit: float = 0.0, shared_limit: float | None = None,
-                 init: str = "normal", gated: bool = True) -> None:
+                 init: str = "normal", gated: bool = True, weigh: str = "output") -> None:
         super().__init__(prefix)
         if not 0 < top <= n_experts:
             raise ValueError(f"top {top} must lie in 1..n_experts ({n_experts})")
@@ -60,6 +65,11 @@ class RoutedExperts(FeedForward):
             count, keep = groups
             if n_experts % count or not 0 < keep <= count or keep * (n_experts // count) < top:
                 raise ValueError(f"groups {groups!r} do not fit {n_experts} experts with {top} choices")
+        if weigh not in ("output", "input"):
+            raise ValueError(f"weigh {weigh!r}: output or input")
+        if weigh == "input" and shared_inner is not None and shared_gate:
+            raise ValueError("a gated shared expert beside experts whose input is weighed is not built")
+        self.weigh = weigh
         self.scoring, self.route_scale, self.has_correction = scoring, float(route_scale), bool(correction)
         self.groups = None if groups is None else (int(groups[0]), int(groups[1]))
         self.activation, self.limit = activation, float(limit)
@@ -69,10 +79,13 @@ class RoutedExperts(FeedForward):
         self.width, self.n_experts, self.top, self.inner = width, n_experts, top, inner
         self.shared_inner = shared_inner
         self.gated = bool(gated)
-        # a plain shared expert as experts that every token uses (see the module's description)
-        self.always = 0 if gated or shared_inner is None else -(-shared_inner // inner)
-        self.returns_output = not gated
         self.shared_gate = bool(shared_gate) and shared_inner is not None
+        # the scores of a plain router: what takes experts that every token uses among the chosen ones
+        self.plain_router = not self.has_correction and self.groups is None
+        # a shared expert as experts that every token uses (see the module's description)
+        folded = not gated or (self.plain_router and not self.shared_gate and activation == "silu")
+        self.always = -(-shared_inner // inner) if folded and shared_inner is not None else 0
+        self.returns_output = folded
         self.router = self.w_in = self.w_out = None
         self.shared_in = self.shared_out = self.shared_gate_weight = None
 
@@ -105,43 +118,38 @@ class RoutedExperts(FeedForward):
         self.correction = tensors.get(p + "correction") if self.has_correction else None
         if self.shared_gate:
             self.shared_gate_weight = tensors[p + "shared.sg"].reshape(-1).contiguous()
-        if not self.gated:
-            ups = [tensors[f"{p}e{e}.up"] for e in range(self.n_experts)]
-            downs = [tensors[f"{p}e{e}.down"] for e in range(self.n_experts)]
-            for first in range(0, self.always * self.inner, self.inner):
-                up = tensors[p + "shared.up"][first: first + self.inner]
-                down = tensors[p + "shared.down"][:, first: first + self.inner]
-                fill = self.inner - up.shape[0]
-                ups.append(torch.nn.functional.pad(up, (0, 0, 0, fill)))
-                downs.append(torch.nn.functional.pad(down, (0, fill)))
-            self.w_in, self.w_out = torch.stack(ups).contiguous(), torch.stack(downs).contiguous()
-            return
-        self.w_in = torch.stack([torch.cat([tensors[f"{p}e{e}.gate"], tensors[f"{p}e{e}.up"]], dim=0)
-                                 for e in range(self.n_experts)]).contiguous()
-        self.w_out = torch.stack([tensors[f"{p}e{e}.down"] for e in range(self.n_experts)]).contiguous()
-        if self.shared_inner is not None:
+        kinds = ("gate", "up") if self.gated else ("up",)
+        ins = [torch.cat([tensors[f"{p}e{e}.{kind}"] for kind in kinds]) for e in range(self.n_experts)]
+        downs = [tensors[f"{p}e{e}.down"] for e in range(self.n_experts)]
+        for first in range(0, self.always * self.inner, self.inner):
+            part = slice(first, first + self.inner)
+            down = tensors[p + "shared.down"][:, part]
+            fill = self.inner - down.shape[1]
+            ins.append(torch.cat([torch.nn.functional.pad(tensors[f"{p}shared.{kind}"][part], (0, 0, 0, fill)) for kind in kinds]))
+            downs.append(torch.nn.functional.pad(down, (0, fill)))
+        self.w_in, self.w_out = torch.stack(ins).contiguous(), torch.stack(downs).contiguous()
+        if self.shared_inner is not None and not self.always:
             self.shared_in = torch.cat([tensors[p + "shared.gate"], tensors[p + "shared.up"]], dim=0).contiguous()
             self.shared_out = tensors[p + "shared.down"]
 
     def forward(self, ctx, y, residual32):
         ops = ctx.ops
-        if not self.gated:
-            ids, weights, _ = ops.moe_route(y, self.router, self.shared_gate_weight, ctx.positions, self.top, always=self.always)
-            if residual32 is None:
-                return ops.moe_experts(y, ids, weights, self.w_in, self.w_out, activation=self.activation, gated=False)
-            ops.moe_experts_residual(y, ids, weights, self.w_in, self.w_out, residual32, activation=self.activation, gated=False)
-            return None
-        if self.scoring == "softmax_top" and not self.has_correction and self.groups is None:
-            ids, weights, gate = ops.moe_route(y, self.router, self.shared_gate_weight, ctx.positions, self.top)
-            if self.route_scale != 1.0:
-                ops.scale_(weights, self.route_scale)
+        extra = {} if self.gated else {"gated": False}
+        if self.activation != "silu":
+            extra.update(activation=self.activation, limit=self.limit)
+        if self.weigh == "input":
+            extra["weigh_input"] = True
+        if self.plain_router:
+            ids, weights, gate = ops.moe_route(y, self.router, self.shared_gate_weight, ctx.positions, self.top,
+                                               always=self.always, scoring=self.scoring, scale=self.route_scale)
         else:
             ids, weights, gate = ops.moe_route_scored(y, self.router, self.shared_gate_weight, ctx.positions, self.top,
                                                       self.scoring, self.correction, self.groups, self.route_scale)
-        plain = self.activation == "silu"
-        ops.moe_experts_residual(y, ids, weights, self.w_in, self.w_out, residual32,
-                                 **({} if plain else {"activation": self.activation, "limit": self.limit}))
-        if self.shared_inner is not None:
+        if residual32 is None:
+            return ops.moe_experts(y, ids, weights, self.w_in, self.w_out, **extra)
+        ops.moe_experts_residual(y, ids, weights, self.w_in, self.w_out, residual32, **extra)
+        if self.shared_inner is not None and not self.always:
+            plain = self.activation == "silu"
             # the shared expert is an ordinary gated unit over all tokens: the projection kernels
             # serve it; its per-token gate rides on the hidden features (W (g h) = g (W h))
             hidden = ops.glu(ops.linear(y, self.shared_in, None, "none", ctx.act_dtype), gate,

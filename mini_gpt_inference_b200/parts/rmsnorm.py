@@ -13,6 +13,7 @@ from .spec import TensorSpec
 @register_norm("rmsnorm")
 class RMSNorm(Norm):
     graph_safe = True      # launches kernels only; nothing is decided on the host per step
+    chains = True
 
     def __init__(self, prefix: str, width: int, eps: float, offset: float = 0.0,
                  weight_name: str | None = None, optional: bool = False) -> None:
@@ -32,10 +33,13 @@ class RMSNorm(Norm):
     def forward(self, ctx, x32):
         return ctx.ops.rmsnorm(x32, self.weight, self.eps, self.offset, ctx.act_dtype)
 
-    def add_normed(self, ctx, y32, residual32, clear=False, scale=1.0, rows_dtype=None):
+    def add_normed(self, ctx, y32, residual32, clear=False, scale=1.0, rows_dtype=None, then=None):
         """``residual32 += scale * norm(y32)`` in 32-bit, in place: the norm behind a sublayer.  ``clear``: ``y32`` is left
         as zeros (a buffer that the next sublayer adds into).  With ``rows_dtype`` the new stream is also returned in
-        that type."""
+        that type; with ``then`` (another of these norms) that norm of the new stream is, in the compute dtype."""
+        if then is not None:
+            return ctx.ops.norm_add(residual32, y32, self.weight, self.eps, self.offset, norm_scale=scale, clear=clear,
+                                    rows_dtype=ctx.act_dtype, then=(then.weight, then.eps, then.offset))
         return ctx.ops.norm_add(residual32, y32, self.weight, self.eps, self.offset, norm_scale=scale, clear=clear,
                                 rows_dtype=rows_dtype)
 

@@ -87,7 +87,7 @@ class TorchOps:
 
     # ---- what the second architecture adds (same conventions as the CUDA kernel set) ---------------
     def head_prepare(self, proj, n_head, n_kv_head, head_dim, v_dim, q_off, k_off, v_off, unit_norm, eps,
-                     cache, slots, positions, v_other=None, blend=None, q_gain=None, k_gain=None):
+                     cache, slots, positions, v_other=None, blend=None, q_gain=None, k_gain=None, q_temperature=None):
         n = proj.shape[0]
         live = positions >= 0
 
@@ -101,7 +101,12 @@ class TorchOps:
         if v_other is not None:
             v = (1.0 - blend[0]) * v + blend[0] * v_other.float()
         v = v.reshape(n, n_kv_head, v_dim)
-        proj[live, q_off: q_off + n_head * head_dim] = unit(q, q_gain)[live].reshape(int(live.sum()), -1).to(proj.dtype)
+        q = unit(q, q_gain)
+        if q_temperature is not None:
+            coef, every = q_temperature
+            steps = torch.floor((positions.clamp(min=0).double() + 1) / every)
+            q = q * (1 + coef * torch.log(steps + 1)).float()[:, None, None]
+        proj[live, q_off: q_off + n_head * head_dim] = q[live].reshape(int(live.sum()), -1).to(proj.dtype)
         if cache is not None and cache.writes:
             keep = live & (slots >= 0)
             page, off = slots[keep].long() // cache.page_tokens, slots[keep].long() % cache.page_tokens
@@ -122,7 +127,7 @@ class TorchOps:
             lo = 0 if cache.window is None else max(0, p - cache.window + 1)
             if block:
                 lo = max(lo, p // block * block)
-            keys = torch.arange(lo, p + 1)
+            keys = torch.cat([torch.arange(min(lo, getattr(cache, "keep_first", 0))), torch.arange(lo, p + 1)])
             pages = table[r, keys // pt]
             assert (pages >= 0).all(), "attention reads a page that is not there"
             k = cache.k_pages[pages, :, keys % pt].float()
@@ -145,10 +150,10 @@ class TorchOps:
             out = out * torch.sigmoid(gate.float())
         return out.to(q.dtype)
 
-    def moe_route(self, y, router_weight, gate_weight, positions, top, always=0):
+    def moe_route(self, y, router_weight, gate_weight, positions, top, always=0, scoring="softmax_top", scale=1.0):
         z = y.float() @ router_weight.float().T
-        vals, ids = torch.topk(z, top, dim=-1)
-        weights = torch.softmax(vals, dim=-1)
+        vals, ids = torch.topk(torch.sigmoid(z) if scoring == "sigmoid" else z, top, dim=-1)
+        weights = scale * (vals if scoring == "sigmoid" else torch.softmax(vals, dim=-1))
         gate = torch.sigmoid(y.float() @ gate_weight.float()) if gate_weight is not None else None
         if always:
             extra = torch.arange(z.shape[1], z.shape[1] + always).expand(len(z), always)
@@ -180,20 +185,21 @@ class TorchOps:
             return z * torch.sigmoid(z)
         raise ValueError(activation)
 
-    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0, gated=True):
+    def moe_experts_residual(self, y, ids, weights, w_in, w_out, residual32, activation="silu", limit=0.0, gated=True,
+                             weigh_input=False):
         inner = w_out.shape[2]
         for t in range(y.shape[0]):
             for k in range(ids.shape[1]):
                 e = int(ids[t, k])
                 if e < 0:
                     continue
-                a = w_in[e].float() @ y[t].float()
+                a = w_in[e].float() @ y[t].float() * (weights[t, k] if weigh_input else 1.0)
                 hidden = self._gated(a[:inner], a[inner:], activation, limit) if gated else self._plain(a, activation)
-                residual32[t] += weights[t, k] * (w_out[e].float() @ hidden.to(y.dtype).float())
+                residual32[t] += (1.0 if weigh_input else weights[t, k]) * (w_out[e].float() @ hidden.to(y.dtype).float())
 
-    def moe_experts(self, y, ids, weights, w_in, w_out, activation="silu", limit=0.0, gated=True):
+    def moe_experts(self, y, ids, weights, w_in, w_out, activation="silu", limit=0.0, gated=True, weigh_input=False):
         out = torch.zeros(y.shape[0], w_out.shape[1])
-        self.moe_experts_residual(y, ids, weights, w_in, w_out, out, activation, limit, gated)
+        self.moe_experts_residual(y, ids, weights, w_in, w_out, out, activation, limit, gated, weigh_input)
         return out
 
     def moe_route_scored(self, y, router_weight, gate_weight, positions, top, scoring, correction, groups, scale):
@@ -463,6 +469,15 @@ class TorchOps:
             cache.k_pages[page, 0, off] = torch.cat([c, shared], dim=-1)[keep].to(cache.k_pages.dtype)
         return q.reshape(n, -1).to(proj.dtype)
 
+    def latent_pair_prepare(self, proj, q_off, q_rank, q_gain, low_off, rank, gain, eps, cache, slots, positions):
+        def normed(off, size, weight):
+            c = proj[:, off: off + size].float()
+            return c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * weight
+        keep = (positions >= 0) & (slots >= 0)
+        page, off = slots[keep].long() // cache.page_tokens, slots[keep].long() % cache.page_tokens
+        cache.k_pages[page, 0, off] = normed(low_off, rank, gain)[keep].to(cache.k_pages.dtype)
+        return normed(q_off, q_rank, q_gain).to(proj.dtype)
+
     def head_linear(self, x, x_off, x_head, weight, rows_are_inputs, n_head, n_in, n_out, gate=None, out=None, out_off=0,
                     out_head=None):
         n = x.shape[0]
@@ -471,7 +486,7 @@ class TorchOps:
         w = weight.float().reshape(n_head, n_in, n_out) if rows_are_inputs else weight.float().reshape(n_head, n_out, n_in).transpose(1, 2)
         y = torch.einsum("nhi,hio->nho", xs, w)
         if gate is not None:
-            y = y * torch.sigmoid(gate.float().reshape(n, n_head, n_out))
+            y = y * torch.sigmoid(gate.float().reshape(n, n_head, -1))           # one number per output, or per head
         if out is None:
             return y.reshape(n, n_head * n_out).to(x.dtype)
         out_head = n_out if out_head is None else out_head
@@ -573,7 +588,7 @@ class TorchOps:
         return out
 
     def norm_add(self, residual32, y32, weight, eps, offset=0.0, center=False, norm_scale=1.0, other32=None, scale=1.0,
-                 other_scale=1.0, clear=False, rows_dtype=None):
+                 other_scale=1.0, clear=False, rows_dtype=None, then=None):
         y = scale * y32 if other32 is None else scale * y32 + other_scale * other32
         if center:
             y = y - y.mean(-1, keepdim=True)
@@ -582,6 +597,8 @@ class TorchOps:
             y32.zero_()
             if other32 is not None:
                 other32.zero_()
+        if then is not None:
+            return self.rmsnorm(residual32, *then, rows_dtype)
         return None if rows_dtype is None else residual32.to(rows_dtype)
 
     def rmsnorm_add(self, residual32, y32, weight, eps, offset=0.0, other32=None, scale=1.0, other_scale=1.0, clear=False):
