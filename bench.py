@@ -32,6 +32,8 @@ four; then the kinds mixed) beside Zenedra's closest layers at equal sizes.
 kinds mixed with a loop and the per-layer token input) beside Zenedra's closest layers at equal sizes.
 ``--only nogatar`` likewise: the Nogatar decoder (layers of one mixer kind each with routed experts, then both kinds
 mixed) beside Nukodra's latent attention, Zenedra's mLSTM and Lunelorn's routed experts at equal sizes.
+``--only vumotar`` likewise: the Vumotar decoder (layers of one attention kind each with routed experts, then the kinds
+mixed) beside Nukodra's windowed attention, Fakilorn's attention and experts and Nogatar's latent attention at equal sizes.
 ``--only designs`` prints a line of its own: the Fakilorn decoder beside this decoder at equal width,
 depth, hidden width and vocabulary (random weights, two sizes): a 2,048-token prompt step, decode
 steps at the headline batch with contexts near 2,048, and the device time of every exported function
@@ -95,7 +97,7 @@ def parse_args():
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--page-tokens", type=int, default=64)
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and prefill")
-    ap.add_argument("--only", choices=["all", "decode", "prefill", "serve", "kernels", "designs", "zenedra", "nukodra", "lunelorn", "nogatar"], default="all",
+    ap.add_argument("--only", choices=["all", "decode", "prefill", "serve", "kernels", "designs", "zenedra", "nukodra", "lunelorn", "nogatar", "vumotar"], default="all",
                     help="a small case for profilers: only the device-timed decode steps, or only "
                          "the 2,048-token prefill (the printed line is then partial); serve: 64 "
                          "requests with prompts of 16 to 512 tokens and 256 generated tokens each "
@@ -790,6 +792,57 @@ def compare_nogatar(args) -> dict:
     return out
 
 
+# ``--only vumotar``: the Vumotar decoder beside the closest layers here at equal width, depth, head count and vocabulary
+# (random weights): Nukodra's attention (a window of 512 and a sink, the same attention kernel; gated dense
+# feed-forwards), Fakilorn's attention with routed experts in every layer (no window, heads of 64, a gated shared
+# expert) and Nogatar's attention over cached latents with the same windows (plain experts).  Vumotar's layers of one kind
+# each: attention with a window of 512 that keeps 16 first tokens, attention whose queries grow, attention over latents of
+# 512 with heads of 128 and queries from a latent of 384, all with routed experts; then the kinds mixed.
+def _vumotar_raw(sz: dict, kinds: list, window) -> dict:
+    heads, kv = sz["heads"], sz["kv_heads"]
+    plain = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 64, "scale": 0.125}
+    mixers = {"attention": {**plain, "mask": {"size": 512, "keep_first": 16}},
+              "attention_2": {**plain, "q_temp": {"coef": 0.1, "every": 512}},
+              "latent_attention": {"heads": heads, "dim": 128, "vdim": 128, "q_rank": 384, "kv_rank": 512, "scale": 128 ** -0.5}}
+    if window:
+        mixers["latent_attention"]["mask"] = {"size": window}
+    routed = {"kind": "moe", "expert": {"ff": sz["expert_ff"]}, "router": {"experts": sz["experts"], "top": sz["top"]},
+              "shared": {"ff": sz["shared_ff"]}}
+    return {"architecture": "Vumotar", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-6},
+            "layers": [{"type": kind, "mixer": dict(mixers[kind]), "mlp": routed} for kind in kinds]}
+
+
+def compare_vumotar(args) -> dict:
+    import torch
+
+    from mini_gpt_inference_b200 import FakilornConfig, NogatarConfig, NukodraConfig, VumotarConfig
+    from mini_gpt_inference_b200.kernels.ops import default_ops
+
+    ops = default_ops("cuda:0")
+    batch, context, prompt_len = args.batch, 2048, PREFILL_TOKENS
+    flush = torch.empty(256 * 1024 * 1024, dtype=torch.uint8, device="cuda:0")
+    out = {"impl": "ours", "partial": "vumotar beside nukodra, fakilorn and nogatar", "dtype": args.dtype, "batch": batch,
+           "context": context, "prompt": prompt_len, "rows": []}
+    for size_name, sz in DESIGN_SIZES.items():
+        n = sz["layers"]
+        fakilorn = _fakilorn_raw(sz, 64, 64, True)
+        routed = fakilorn["layers"][1]["mlp"]
+        fakilorn["layers"] = [{**layer, "mlp": routed} for layer in fakilorn["layers"]]
+        mixed = (["latent_attention", "attention", "attention_2", "latent_attention"] * n)[:n]
+        for name, cfg in (
+                ("nukodra {} attention, window 512, dense", NukodraConfig.from_dict(_nukodra_raw(sz, ["attention"] * n, None))),
+                ("fakilorn {} attention, experts", FakilornConfig.from_dict(fakilorn)),
+                ("nogatar {} latent attention, experts", NogatarConfig.from_dict(_nogatar_raw(sz, ["latent_attention"] * n, None))),
+                ("nogatar {} latent attention, window 512, experts", NogatarConfig.from_dict(_nogatar_raw(sz, ["latent_attention"] * n, 512))),
+                ("vumotar {} attention, window 512 and 16 kept, experts", VumotarConfig.from_dict(_vumotar_raw(sz, ["attention"] * n, None))),
+                ("vumotar {} attention_2, experts", VumotarConfig.from_dict(_vumotar_raw(sz, ["attention_2"] * n, None))),
+                ("vumotar {} latent attention, experts", VumotarConfig.from_dict(_vumotar_raw(sz, ["latent_attention"] * n, None))),
+                ("vumotar {} latent attention, window 512, experts", VumotarConfig.from_dict(_vumotar_raw(sz, ["latent_attention"] * n, 512))),
+                ("vumotar {} mixed, window 512, experts", VumotarConfig.from_dict(_vumotar_raw(sz, mixed, 512)))):
+            out["rows"].append(_measure_design(args, ops, flush, name.format(size_name), cfg, batch, context, prompt_len))
+    return out
+
+
 def check_decode_logits(args) -> dict:
     """Outside every timed region: the decode step that the benchmark times (batch 8, contexts of
     2,048, the replayed graph) is run once on fixed tokens and its logits are compared with rows
@@ -859,6 +912,8 @@ def run_ours(args) -> dict:
         return compare_lunelorn(args)
     if args.only == "nogatar":
         return compare_nogatar(args)
+    if args.only == "vumotar":
+        return compare_vumotar(args)
     if args.only == "decode":
         cfg, windows, launches, mean_ctx, clocks = device_decode(args, args.batch, args.steps, args.warmup,
                                                                  min_seconds=0.0)
